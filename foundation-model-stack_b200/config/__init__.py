@@ -1,6 +1,6 @@
 from .model_config import ModelConfig
 from .specs import (BlockSpec, DecoderSpec, EmbeddingSpec, FeedForwardSpec, LayerCall, MixerSpec, NormSpec,
-                    PositionSpec)
+                    PositionSpec, TokenSideSpec)
 
 __all__ = ["ModelConfig", "BlockSpec", "DecoderSpec", "EmbeddingSpec", "FeedForwardSpec", "LayerCall", "MixerSpec",
-           "NormSpec", "PositionSpec"]
+           "NormSpec", "PositionSpec", "TokenSideSpec"]

@@ -67,6 +67,18 @@ class FeedForwardSpec:
 
 
 @dataclasses.dataclass(frozen=True)
+class TokenSideSpec:
+    """What a layer adds for the tokens themselves after its sublayers (``fms_b200.parts.token_side``): ``dim`` values of
+    the token's row of the layer's table, gated by the stream, projected to ``width`` and normed."""
+
+    vocab_size: int
+    dim: int
+    width: int
+    eps: float
+    activation: str = "gelu-tanh"
+
+
+@dataclasses.dataclass(frozen=True)
 class BlockSpec:
     """One layer: its norms, mixer and feed-forward and their arrangement, which names the block class in the
     registry (``fms_b200.parts.register_block``).  ``arrangement == "pre_norm"``:
@@ -75,7 +87,8 @@ class BlockSpec:
     ``alpha`` in ``options``.  ``arrangement == "sandwich"``: every sublayer's output is
     normed once more before it is added, x += norm1b(mixer(norm1(x))); x += norm2b(feed_forward(norm2(x))); the two
     further norms are ``mixer_post_norm`` and ``feed_forward_post_norm``, and a layer without a feed-forward
-    (``feed_forward is None``) ends after its mixer.  The names are those under which the layer's
+    (``feed_forward is None``) ends after its mixer.  ``arrangement == "parallel_joint"``: both sublayers read one norm,
+    x += mixer(norm1(x)) + feed_forward(norm1(x)), through one joint projection, and ``token_side`` (optional) follows.  The names are those under which the layer's
     parts appear in weight names (``ln``, ``attn``, ``ff_ln``, ``ff_sub_layer`` for Llama); ``post_names`` those of
     the two further norms."""
 
@@ -89,6 +102,7 @@ class BlockSpec:
     mixer_post_norm: Optional[NormSpec] = None
     feed_forward_post_norm: Optional[NormSpec] = None
     post_names: Tuple[str, str] = ("post_ln", "ff_post_ln")
+    token_side: Optional[TokenSideSpec] = None
     # the layer has no tensors of its own: it runs with the parts (mixer, feed-forward, norms) of that earlier layer,
     # whose spec its own equals, and with a cache entry or state of its own
     weights_of: Optional[int] = None
@@ -111,6 +125,7 @@ class LayerCall:
 @dataclasses.dataclass(frozen=True)
 class EmbeddingSpec:
     """How token ids become the first rows of the residual stream.  ``kind == "table"``: a row of the token table.
+    ``kind == "table_and_positions"``: that row plus a row of a table of learned positions (option ``positions``: how many).
     ``kind == "pair_hash"``: that row plus a row of a second table, found by hashing the token with the one before it:
     row (previous * mul_prev + token * mul_cur) mod buckets, and row ``buckets`` (the table has buckets + 1 rows) for
     a sequence's first token; options ``buckets``, ``mul_prev``, ``mul_cur``, ``name`` (the second table's tensor)."""

@@ -43,7 +43,7 @@ template <> __device__ __forceinline__ void load_vec<float>(const float* p, floa
 }
 
 struct AttnArgs {
-  const void* q;        // [tokens, nheads * HD]
+  const void* q;        // token t, head h at t * q_stride + h * HD
   void* out;            // [tokens, nheads * HD]
   const void* keys;     // cache
   const void* values;
@@ -64,6 +64,10 @@ struct AttnArgs {
   // query sees the keys of its own run only.  softcap > 0: a score is softcap * tanh(score / softcap) after the scale.
   int chunk;
   float softcap;
+  // [nheads] pairs (r1, r2) float32 or null: what is taken off a score (after the cap) for the distance between query and
+  // key, r1 * ln(1 + r2 * (query position - key position))
+  const float2* distance;
+  long q_stride;  // values from one token's queries to the next's (nheads * HD, or the row of a wider matrix); set by every entry
 };
 
 // The first position that the query at `pos` sees (its last is pos).  It never decreases as pos grows, so a tile of
@@ -82,6 +86,17 @@ __device__ __forceinline__ int first_visible(const AttnArgs& a, int pos) {
 __device__ __forceinline__ float capped_raw(const AttnArgs& a, float raw) {
   const float t = __expf(2.f * raw * (a.scale / a.softcap));
   return (1.f - __fdividef(2.f, t + 1.f)) * (a.softcap / a.scale);
+}
+
+// The distance term in the same units, r' with r' * scale = r1 * ln(1 + r2 * distance): `factor` is r1 * ln(2) / scale
+// (distance_factor), the logarithm the one-instruction base-2 one.  For keys after the query it may be NaN; their
+// scores are masked by selection afterwards.
+__device__ __forceinline__ float2 distance_factor(const AttnArgs& a, int head) {
+  const float2 r = a.distance[head];
+  return make_float2(r.x * (0.69314718055994531f / a.scale), r.y);
+}
+__device__ __forceinline__ float distance_raw(float2 factor, int distance) {
+  return factor.x * __log2f(fmaf(factor.y, (float)distance, 1.f));
 }
 
 // The cache block that holds key block kb of the sequence in `slot`; negative: none (a block given back behind a
@@ -122,7 +137,7 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(AttnArgs a, const int
   for (int i = tid; i < TQ * HD; i += 128) {
     const int rr = i / HD, d = i - rr * HD;
     qs[rr * (HD + 1) + d] =
-        rr < rows_here ? to_f32(q[(size_t)(row_begin + r0 + rr) * a.nheads * HD + (size_t)head * HD + d]) : 0.f;
+        rr < rows_here ? to_f32(q[(size_t)(row_begin + r0 + rr) * a.q_stride + (size_t)head * HD + d]) : 0.f;
   }
   const int p_first = len_before + r0;
   const int p_last = p_first + rows_here - 1;
@@ -131,6 +146,7 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(AttnArgs a, const int
   const int kb_lo = first_visible(a, p_first) / BLK;
   const int kb_hi = p_last / BLK;
   const int my_first = first_visible(a, my_pos);
+  const float2 dist = a.distance ? a.distance[head] : make_float2(0.f, 0.f);
 
   float m = -INFINITY, l = 0.f;
   float acc[HD / 8];
@@ -172,6 +188,7 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(AttnArgs a, const int
       for (int d = 0; d < HD; ++d) dot = fmaf(qr[d], kr[d], dot);
       const bool visible = row_ok && kpos <= my_pos && kpos >= my_first;
       s[i] = visible ? (a.softcap > 0.f ? a.softcap * tanhf(dot * a.scale / a.softcap) : dot * a.scale) : -INFINITY;
+      if (a.distance && visible) s[i] -= dist.x * log1pf(dist.y * (float)(my_pos - kpos));
       tile_max = fmaxf(tile_max, s[i]);
     }
     tile_max = fmaxf(tile_max, __shfl_xor_sync(0xffffffffu, tile_max, 1));
@@ -245,7 +262,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnArgs a, float* __r
   if (k_lo >= k_hi) return;
   const int slot = a.slots[seq];
   const int row = a.first_row[seq];
-  const T* q = (const T*)a.q + (size_t)row * a.nheads * HD + (size_t)(kvh * group + g0) * HD;
+  const T* q = (const T*)a.q + (size_t)row * a.q_stride + (size_t)(kvh * group + g0) * HD;
   const T* kc = (const T*)a.keys;
   const T* vc = (const T*)a.values;
 
@@ -291,7 +308,14 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnArgs a, float* __r
       for (int g = 0; g < GC; ++g) {
         const float other = __shfl_xor_sync(0xffffffffu, dot[g], 1);
         const float sc = dot[g] + other;  // the scale is in the queries
-        if (half == 0) ss[g][key_of] = valid ? (a.softcap > 0.f ? a.softcap * tanhf(sc / a.softcap) : sc) : -INFINITY;
+        if (half == 0) {
+          float s = valid ? (a.softcap > 0.f ? a.softcap * tanhf(sc / a.softcap) : sc) : -INFINITY;
+          if (a.distance && valid && g < ng) {
+            const float2 dist = a.distance[kvh * group + g0 + g];
+            s -= dist.x * log1pf(dist.y * (float)(pos - kpos));
+          }
+          ss[g][key_of] = s;
+        }
       }
     }
     __syncthreads();
@@ -451,6 +475,14 @@ int check_args(const char* what, int nheads, int kvheads, int head_dim, int bloc
   return 0;
 }
 
+// the kernels read queries 16 bytes at a time
+int check_queries(const void* q, int dtype, long q_stride, int nheads) {
+  const long item = dtype == FMS_BF16 ? 2 : 4;
+  if (q_stride < (long)nheads * HD || (q_stride * item) % 16 || (uintptr_t)q % 16)
+    return fms_fail("attention: queries %ld values apart for %d heads of %d, or not on 16 bytes", q_stride, nheads, HD);
+  return 0;
+}
+
 int check_mask(const char* what, int window, int chunk, float softcap) {
   if (window < 0 || chunk < 0 || (window > 0 && chunk > 0))
     return fms_fail("%s: window %d, chunk %d: one of them at most, neither negative", what, window, chunk);
@@ -587,12 +619,13 @@ static int attention_prefill(const void* q, void* out, int dtype, const void* ke
                              const int* first_row, const int* len_after, const int* tiles, int n_tiles,
                              int nheads, int kvheads, int head_dim, float scale, int window, int pool_blocks,
                              int table_rows, int* error_flag, const float* sink, cudaStream_t stream, int chunk = 0,
-                             float softcap = 0.f) {
+                             float softcap = 0.f, const float* distance = nullptr, long q_stride = 0) {
   if (n_tiles <= 0) return 0;
   if (check_args("attention_prefill", nheads, kvheads, head_dim, block_tokens)) return 1;
   if (check_mask("attention_prefill", window, chunk, softcap)) return 1;
   AttnArgs a{q, out, keys, values, table, table_stride, slots, first_row, len_after, nheads, kvheads, scale, window,
-             table_rows, pool_blocks, sink, chunk, softcap};
+             table_rows, pool_blocks, sink, chunk, softcap, (const float2*)distance, q_stride > 0 ? q_stride : (long)nheads * HD};
+  if (check_queries(q, dtype, a.q_stride, nheads)) return 1;
   if (nheads > 65535) return fms_fail("attention_prefill: %d heads", nheads);
   if (!(scale > 0.f)) return fms_fail("attention_prefill: the scale of the scores is %g; it must be positive", (double)scale);
 #if FMS_ATTENTION_TC
@@ -664,16 +697,17 @@ FMS_API int fms_attention_prefill_sink(const void* q, void* out, int dtype, cons
 }
 
 // The same with, each of them optional, a sink per head (null: none), keys seen in runs of `chunk` positions (0: all
-// keys, or the window's) and capped scores (softcap 0: none).
+// keys, or the window's), capped scores (softcap 0: none) and a distance term ([nheads][2] float32: r1 and r2; null: none).
+// q_stride: values from one token's queries to the next's (0: nheads * head size).
 FMS_API int fms_attention_prefill_masked(const void* q, void* out, int dtype, const void* keys, const void* values,
                                          const int* table, int table_stride, int block_tokens, const int* slots,
                                          const int* first_row, const int* len_after, const int* tiles, int n_tiles,
                                          int nheads, int kvheads, int head_dim, float scale, int window, int pool_blocks,
                                          int table_rows, int* error_flag, const float* sink, int chunk, float softcap,
-                                         cudaStream_t stream) {
+                                         const float* distance, long q_stride, cudaStream_t stream) {
   return attention_prefill(q, out, dtype, keys, values, table, table_stride, block_tokens, slots, first_row, len_after,
                            tiles, n_tiles, nheads, kvheads, head_dim, scale, window, pool_blocks, table_rows, error_flag,
-                           sink, stream, chunk, softcap);
+                           sink, stream, chunk, softcap, distance, q_stride);
 }
 
 // part_o: float [seqs, nheads, n_splits, HD]; part_ml: float [seqs, nheads, n_splits, 2]; both scratch.
@@ -693,7 +727,7 @@ FMS_API int fms_attention_decode(const void* q, void* out, int dtype, const void
   if (check_args("attention_decode", nheads, kvheads, head_dim, block_tokens)) return 1;
   if (!(scale > 0.f)) return fms_fail("attention_decode: the scale of the scores is %g; it must be positive", (double)scale);
   AttnArgs a{q, out, keys, values, table, table_stride, slots, first_row, len_after, nheads, kvheads, scale, window,
-             table_rows, pool_blocks, nullptr};
+             table_rows, pool_blocks, nullptr, 0, 0.f, nullptr, (long)nheads * HD};
   return launch_decode("attention_decode", a, dtype, n_seqs, n_splits, part_o, part_ml, pool_blocks, total_len, work_counter, error_flag, stream);
 }
 
@@ -708,24 +742,27 @@ FMS_API int fms_attention_decode_sink(const void* q, void* out, int dtype, const
   if (check_args("attention_decode", nheads, kvheads, head_dim, block_tokens)) return 1;
   if (!(scale > 0.f)) return fms_fail("attention_decode: the scale of the scores is %g; it must be positive", (double)scale);
   AttnArgs a{q, out, keys, values, table, table_stride, slots, first_row, len_after, nheads, kvheads, scale, window,
-             table_rows, pool_blocks, sink};
+             table_rows, pool_blocks, sink, 0, 0.f, nullptr, (long)nheads * HD};
   return launch_decode("attention_decode", a, dtype, n_seqs, n_splits, part_o, part_ml, pool_blocks, total_len, work_counter, error_flag, stream);
 }
 
 // The same with, each of them optional, a sink per head (null: none), keys seen in runs of `chunk` positions (0: all
-// keys, or the window's) and capped scores (softcap 0: none).
+// keys, or the window's), capped scores (softcap 0: none) and a distance term ([nheads][2] float32: r1 and r2; null: none).
+// q_stride: values from one token's queries to the next's (0: nheads * head size).
 FMS_API int fms_attention_decode_masked(const void* q, void* out, int dtype, const void* keys, const void* values,
                                         const int* table, int table_stride, int block_tokens, const int* slots,
                                         const int* first_row, const int* len_after, int n_seqs, int n_splits, float* part_o,
                                         float* part_ml, int nheads, int kvheads, int head_dim, float scale, int window,
                                         int pool_blocks, int table_rows, long total_len, int* work_counter, int* error_flag,
-                                        const float* sink, int chunk, float softcap, cudaStream_t stream) {
+                                        const float* sink, int chunk, float softcap, const float* distance, long q_stride,
+                                        cudaStream_t stream) {
   if (n_seqs <= 0) return 0;
   if (check_args("attention_decode", nheads, kvheads, head_dim, block_tokens)) return 1;
   if (check_mask("attention_decode", window, chunk, softcap)) return 1;
   if (!(scale > 0.f)) return fms_fail("attention_decode: the scale of the scores is %g; it must be positive", (double)scale);
   AttnArgs a{q, out, keys, values, table, table_stride, slots, first_row, len_after, nheads, kvheads, scale, window,
-             table_rows, pool_blocks, sink, chunk, softcap};
+             table_rows, pool_blocks, sink, chunk, softcap, (const float2*)distance, q_stride > 0 ? q_stride : (long)nheads * HD};
+  if (check_queries(q, dtype, a.q_stride, nheads)) return 1;
   return launch_decode("attention_decode", a, dtype, n_seqs, n_splits, part_o, part_ml, pool_blocks, total_len, work_counter, error_flag, stream);
 }
 
@@ -784,6 +821,7 @@ FMS_API int fms_attention_decode_no_alloc(const void* q, void* out, int dtype, c
   if (scratch == nullptr) return 1;
   float* part_o = scratch;                  // [seqs, nheads, n_splits, HD]
   float* part_ml = scratch + entries * HD;  // [seqs, nheads, n_splits, 2]
-  AttnArgs a{q, out, keys, values, table, table_stride, slots, first_row, len_after, nheads, kvheads, scale, window, 0, 0, nullptr};
+  AttnArgs a{q, out, keys, values, table, table_stride, slots, first_row, len_after, nheads, kvheads, scale, window, 0, 0, nullptr, 0, 0.f, nullptr,
+             (long)nheads * HD};
   return launch_decode("attention_decode_no_alloc", a, dtype, n_seqs, n_splits, part_o, part_ml, 0, 0, nullptr, nullptr, stream);
 }

@@ -152,7 +152,7 @@ __global__ void __launch_bounds__(NW * 32, WK == 32 ? 16 / NW : 12 / NW)
   const int kstart = first_visible(a, pos);
   const int k_lo = max(kstart, split * SPLIT), k_hi = min(len, (split + 1) * SPLIT);
   if (k_lo >= k_hi) return;
-  const __nv_bfloat16* q = (const __nv_bfloat16*)a.q + (size_t)first_row * a.nheads * HD +
+  const __nv_bfloat16* q = (const __nv_bfloat16*)a.q + (size_t)first_row * a.q_stride +
                            (size_t)(kvh * group + g0) * HD;
   const __nv_bfloat16* kc = (const __nv_bfloat16*)a.keys;
   const __nv_bfloat16* vc = (const __nv_bfloat16*)a.values;
@@ -182,6 +182,13 @@ __global__ void __launch_bounds__(NW * 32, WK == 32 ? 16 / NW : 12 / NW)
   for (int j = 0; j < HD / 16; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};  // of heads 2 c and 2 c + 1; maximum in units of log2
   const float scale2 = a.scale * LOG2E;  // scores are kept times log2(e): exp(x) = exp2(x log2 e)
+
+  float2 dist[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};  // of heads 2 c and 2 c + 1
+  if (a.distance) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h)
+      if (2 * c + h < ng) dist[h] = distance_factor(a, kvh * group + g0 + 2 * c + h);
+  }
 
   bool first_block = true;
   constexpr int WT = WK / 16;  // mma tiles of 16 keys a piece
@@ -252,6 +259,12 @@ __global__ void __launch_bounds__(NW * 32, WK == 32 ? 16 / NW : 12 / NW)
       for (int t = 0; t < WT; ++t)
 #pragma unroll
         for (int e = 0; e < 4; ++e) st[t][e] = capped_raw(a, st[t][e]);
+    }
+    if (a.distance) {
+#pragma unroll
+      for (int t = 0; t < WT; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) st[t][e] -= distance_raw(dist[e & 1], pos - (first + 16 * t + g + 8 * (e >> 1)));
     }
     if (!whole) {
 #pragma unroll
@@ -426,9 +439,16 @@ __global__ void __launch_bounds__(PF_WARPS * 32, HD <= 128 ? 3 : 1) attn_prefill
     row_ok[h] = pi < pos_here && gi < ng;
     row_pos[h] = p_first + pi;
     row_first[h] = first_visible(a, row_pos[h]);
-    const size_t at = ((size_t)(row_begin + r0 + (row_ok[h] ? pi : 0)) * a.nheads + kvh * group + g0 + (row_ok[h] ? gi : 0)) * HD;
-    qrow[h] = q + at;
-    orow[h] = (__nv_bfloat16*)a.out + at;
+    const size_t token = row_begin + r0 + (row_ok[h] ? pi : 0);
+    const int head = kvh * group + g0 + (row_ok[h] ? gi : 0);
+    qrow[h] = q + token * a.q_stride + (size_t)head * HD;
+    orow[h] = (__nv_bfloat16*)a.out + (token * a.nheads + head) * HD;
+  }
+  float2 dist[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
+  if (a.distance) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h)
+      if (row_ok[h]) dist[h] = distance_factor(a, kvh * group + g0 + (warp * 16 + g + 8 * h) % gh);
   }
   uint32_t qf[HD / 16][4];
 #pragma unroll
@@ -484,6 +504,13 @@ __global__ void __launch_bounds__(PF_WARPS * 32, HD <= 128 ? 3 : 1) attn_prefill
       for (int j = 0; j < 8; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) s[j][e] = capped_raw(a, s[j][e]);
+    }
+    if (a.distance) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          s[j][e] -= distance_raw(dist[e >> 1], row_pos[e >> 1] - (kb * BLK + 8 * j + 2 * c + (e & 1)));
     }
     float tile_max[2] = {-INFINITY, -INFINITY};
 #pragma unroll

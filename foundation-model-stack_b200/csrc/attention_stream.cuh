@@ -117,7 +117,7 @@ __global__ void __launch_bounds__((SR_WARPS + 1) * 32, 1)
       }
       if (first_here)
         bulk_copy_g2s(st + 2 * SR_KV_BYTES,
-                      (const __nv_bfloat16*)a.q + ((size_t)a.first_row[seq] * a.nheads + kvh * group + g0) * HD, ng * HD * 2,
+                      (const __nv_bfloat16*)a.q + (size_t)a.first_row[seq] * a.q_stride + (size_t)(kvh * group + g0) * HD, ng * HD * 2,
                       full + s);
     }
   }
@@ -131,6 +131,8 @@ __global__ void __launch_bounds__((SR_WARPS + 1) * 32, 1)
   float o[HD / 16][4];
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   const float scale2 = a.scale * LOG2E;
+  float2 dist[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};  // of heads 2 c and 2 c + 1 of the unit at hand
+  int pos = 0;                                                       // its query's position
   for (int i = 0;; ++i) {
     const int s = i % SR_STAGES;
     if (!mbar_wait(full + s, (uint32_t)(i / SR_STAGES) & 1u)) {
@@ -191,6 +193,18 @@ __global__ void __launch_bounds__((SR_WARPS + 1) * 32, 1)
       for (int t = 0; t < 4; ++t)
 #pragma unroll
         for (int e = 0; e < 4; ++e) st[t][e] = capped_raw(a, st[t][e]);
+    }
+    if (a.distance) {
+      if (first) {
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+          dist[h] = 2 * c + h < ng ? distance_factor(a, kvh * group + g0 + 2 * c + h) : make_float2(0.f, 0.f);
+        pos = a.len_after[seq] - 1;
+      }
+#pragma unroll
+      for (int t = 0; t < 4; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) st[t][e] -= distance_raw(dist[e & 1], pos - (kb * BLK + 16 * t + g + 8 * (e >> 1)));
     }
     if (!whole) {
 #pragma unroll

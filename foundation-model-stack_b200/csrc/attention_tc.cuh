@@ -177,7 +177,7 @@ __global__ void __launch_bounds__(192, 2) attn_prefill_tc_kernel(const __grid_co
     // the query tile: row r, 16-byte piece c of 64-value chunk t at t * 16 KB + r * 128 + ((c ^ (r & 7)) << 4)
     {
       const __nv_bfloat16* q = (const __nv_bfloat16*)a.q +
-                               ((size_t)(row_begin + r0 + (row_ok ? pi : 0)) * a.nheads + kvh * group + g0 + (row_ok ? gi : 0)) * HD;
+                               (size_t)(row_begin + r0 + (row_ok ? pi : 0)) * a.q_stride + (size_t)(kvh * group + g0 + (row_ok ? gi : 0)) * HD;
 #pragma unroll
       for (int c = 0; c < HD / 8; ++c) {
         const uint4 v = row_ok ? *reinterpret_cast<const uint4*>(q + 8 * c) : make_uint4(0, 0, 0, 0);
@@ -187,6 +187,7 @@ __global__ void __launch_bounds__(192, 2) attn_prefill_tc_kernel(const __grid_co
       mbar_arrive(q_ready);
     }
     const float scale2 = a.scale * LOG2E;
+    const float2 dist = a.distance && row_ok ? distance_factor(a, kvh * group + g0 + gi) : make_float2(0.f, 0.f);
     float m_ref = -INFINITY, l = 0.f;  // the exponents are taken against m_ref (base 2); l is the sum of them
     bool ok = true;
     for (int i = 0; i < nblocks && ok; ++i) {
@@ -203,6 +204,10 @@ __global__ void __launch_bounds__(192, 2) attn_prefill_tc_kernel(const __grid_co
       if (a.softcap > 0.f) {
 #pragma unroll
         for (int j = 0; j < BLK; ++j) sc[j] = capped_raw(a, sc[j]);
+      }
+      if (a.distance) {
+#pragma unroll
+        for (int j = 0; j < BLK; ++j) sc[j] -= distance_raw(dist, my_pos - (kb * BLK + j));
       }
       if (!whole) {
 #pragma unroll

@@ -3,8 +3,36 @@
 // All arithmetic is float32; inputs and outputs are float32 or bfloat16.
 #include "common.cuh"
 
+// four consecutive values at once (the pointer aligned to four values)
+__device__ __forceinline__ void ldv4(const float* p, float (&v)[4]) {
+  const float4 t = *reinterpret_cast<const float4*>(p);
+  v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
+}
+__device__ __forceinline__ void ldv4(const __nv_bfloat16* p, float (&v)[4]) {
+  const uint2 t = *reinterpret_cast<const uint2*>(p);
+  v[0] = __uint_as_float(t.x << 16); v[1] = __uint_as_float(t.x & 0xffff0000u);
+  v[2] = __uint_as_float(t.y << 16); v[3] = __uint_as_float(t.y & 0xffff0000u);
+}
+__device__ __forceinline__ void stv4(float* p, const float (&v)[4]) {
+  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+__device__ __forceinline__ void stv4(__nv_bfloat16* p, const float (&v)[4]) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+  uint2 t;
+  t.x = *reinterpret_cast<const uint32_t*>(&a);
+  t.y = *reinterpret_cast<const uint32_t*>(&b);
+  *reinterpret_cast<uint2*>(p) = t;
+}
+
+// up to four sublayer outputs (in the compute dtype; null: not given) with a factor each
+struct NormParts {
+  const void* d[4];
+  float s[4];
+};
+
 // ---------------------------------------------------------------------------------------------------
 // embedding: out[t, :] = scale * float(table[tokens[t], :])    (reference: fms/models/llama.py:332; scale 1)
+// with a table of learned positions also + float(pos_table[positions[t], :]), unscaled
 // ---------------------------------------------------------------------------------------------------
 __device__ __forceinline__ void embed_load8(const float* p, float* v) {
   const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
@@ -22,16 +50,28 @@ __device__ __forceinline__ void embed_load8(const __nv_bfloat16* p, float* v) {
 
 template <typename T>
 __global__ void embed_rows_kernel(const T* __restrict__ table, const int* __restrict__ tokens, float* __restrict__ out,
-                                  int dim, int vocab, float scale, int* __restrict__ error_flag) {
+                                  int dim, int vocab, float scale, int* __restrict__ error_flag, const T* pos_table,
+                                  const int* positions, int n_positions) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
   const int tok = tokens[t];
-  const bool ok = tok >= 0 && tok < vocab;
+  bool ok = tok >= 0 && tok < vocab;
   if (!ok && threadIdx.x == 0 && error_flag) atomicExch(error_flag, 1);
+  const T* place = nullptr;
+  if (pos_table) {
+    const int pos = __ldcg(positions + t);
+    if (pos < 0 || pos >= n_positions) {
+      if (threadIdx.x == 0 && error_flag) atomicExch(error_flag, 32);
+      ok = false;
+    } else {
+      place = pos_table + (size_t)pos * dim;
+    }
+  }
   const T* src = table + (size_t)(ok ? tok : 0) * dim;
   float* dst = out + (size_t)t * dim;
-  if ((dim & 7) == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0 && (reinterpret_cast<uintptr_t>(dst) & 15) == 0) {
+  if ((dim & 7) == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0 && (reinterpret_cast<uintptr_t>(dst) & 15) == 0 &&
+      (reinterpret_cast<uintptr_t>(place) & 15) == 0) {
     // 8 values a thread and step: 16 bytes in for bfloat16 (two loads for float32), two 16-byte stores out
     for (int d = 8 * threadIdx.x; d < dim; d += 8 * blockDim.x) {
       float v[8];
@@ -40,13 +80,37 @@ __global__ void embed_rows_kernel(const T* __restrict__ table, const int* __rest
       if (ok) {
         a = make_float4(scale * v[0], scale * v[1], scale * v[2], scale * v[3]);
         b = make_float4(scale * v[4], scale * v[5], scale * v[6], scale * v[7]);
+        if (place) {
+          embed_load8(place + d, v);
+          a.x += v[0]; a.y += v[1]; a.z += v[2]; a.w += v[3];
+          b.x += v[4]; b.y += v[5]; b.z += v[6]; b.w += v[7];
+        }
       }
       *reinterpret_cast<float4*>(dst + d) = a;
       *reinterpret_cast<float4*>(dst + d + 4) = b;
     }
     return;
   }
-  for (int d = threadIdx.x; d < dim; d += blockDim.x) dst[d] = ok ? scale * to_f32(src[d]) : 0.f;
+  for (int d = threadIdx.x; d < dim; d += blockDim.x) {
+    float v = ok ? scale * to_f32(src[d]) : 0.f;
+    if (ok && place) v += to_f32(place[d]);
+    dst[d] = v;
+  }
+}
+
+// pos_table [n_positions, dim] in the table's dtype, positions [n_tokens]: a position outside the table sets error flag
+// 32 and gives a row of zeros
+FMS_API int fms_embed_rows_at(const void* table, int table_dtype, const int* tokens, float* out, int n_tokens, int dim,
+                              int vocab, float scale, const void* pos_table, const int* positions, int n_positions,
+                              int* error_flag, cudaStream_t stream) {
+  if (n_tokens <= 0) return 0;
+  if (dim <= 0 || vocab <= 0 || n_positions <= 0 || !pos_table || !positions)
+    return fms_fail("embed_rows_at: dim %d, vocab %d, %d positions", dim, vocab, n_positions);
+  const int threads = dim >= 1024 ? 256 : 128;
+  FMS_DISPATCH_DTYPE(table_dtype, T,
+                     fms_launch(embed_rows_kernel<T>, dim3(n_tokens), dim3(threads), 0, stream, (const T*)table, tokens,
+                                out, dim, vocab, scale, error_flag, (const T*)pos_table, positions, n_positions));
+  return fms_launch_status("embed_rows_at");
 }
 
 FMS_API int fms_embed_rows(const void* table, int table_dtype, const int* tokens, float* out, int n_tokens, int dim,
@@ -56,7 +120,7 @@ FMS_API int fms_embed_rows(const void* table, int table_dtype, const int* tokens
   const int threads = dim >= 1024 ? 256 : 128;
   FMS_DISPATCH_DTYPE(table_dtype, T,
                      fms_launch(embed_rows_kernel<T>, dim3(n_tokens), dim3(threads), 0, stream, (const T*)table, tokens,
-                                out, dim, vocab, scale, error_flag));
+                                out, dim, vocab, scale, error_flag, (const T*)nullptr, (const int*)nullptr, 0));
   return fms_launch_status("embed_rows");
 }
 
@@ -403,17 +467,18 @@ FMS_API int fms_normed_add_rmsnorm(float* residual, const void* delta, int has_p
 
 // ---------------------------------------------------------------------------------------------------
 // The same step for norms of either kind, each chosen by a mode: 0 none, 1 root mean square, 2 layer norm (the mean is
-// taken off first and the variance is the mean of the squared deviations; no bias).  Gains are float32 vectors of
-// `dim` (a layer scale that multiplies a norm's result is folded into its gain by the caller):
-//   d = post(delta) * post_gain                              post_mode 0: d = delta
-//   x = residual[src] + d                float32; written back to residual unless rows are gathered
-//   out[r] = norm(x) * gain                                   out_mode 0: out[r] = x, the stream in the compute dtype
+// taken off first and the variance is the mean of the squared deviations).  Gains are float32 vectors of `dim` (a layer
+// scale that multiplies a norm's result is folded into its gain by the caller), `bias` one that is added at the end:
+//   d = post(d0) * post_gain                                 post_mode 0: d = s0 d0
+//   x = residual[src] + d + s1 d1 + s2 d2 + s3 d3            (the parts that are given; float32); written back to
+//                                                             residual unless rows are gathered
+//   out[r] = norm(x) * gain + bias                            out_mode 0: out[r] = x, the stream in the compute dtype
 //                                                             (no out pointer: nothing but the sum is wanted)
-// A block per row with the row in registers, NPER values a thread (dim <= NPER * blockDim).
+// A block per row with the row in registers, NPER values a thread (dim <= NPER * blockDim), in runs of VEC neighbours.
 // ---------------------------------------------------------------------------------------------------
-template <int NPER>
-__device__ __forceinline__ void norm_in_registers(float (&v)[NPER], int mode, const float* gain_vec, float eps, int dim,
-                                                  float* scratch) {
+template <int NPER, int VEC>
+__device__ __forceinline__ void norm_in_registers(float (&v)[NPER], int mode, const float* gain_vec, const float* bias,
+                                                  float eps, int dim, float* scratch) {
   if (mode == 0) return;
   float mean = 0.f;
   if (mode == 2) {
@@ -425,23 +490,33 @@ __device__ __forceinline__ void norm_in_registers(float (&v)[NPER], int mode, co
   float ss = 0.f;
 #pragma unroll
   for (int j = 0; j < NPER; ++j) {
-    const int d = threadIdx.x + j * blockDim.x;
+    const int d = (threadIdx.x + (j / VEC) * blockDim.x) * VEC + j % VEC;
     const float c = d < dim ? v[j] - mean : 0.f;
     v[j] = c;
     ss += c * c;
   }
   const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)dim + eps);
 #pragma unroll
-  for (int j = 0; j < NPER; ++j) {
-    const int d = threadIdx.x + j * blockDim.x;
-    if (d < dim) v[j] = v[j] * inv * gain_vec[d];
+  for (int j = 0; j < NPER; j += VEC) {
+    const int d = (threadIdx.x + (j / VEC) * blockDim.x) * VEC;
+    if (d >= dim) continue;
+    if constexpr (VEC == 4) {
+      float g[4], b[4] = {0.f, 0.f, 0.f, 0.f};
+      ldv4(gain_vec + d, g);
+      if (bias) ldv4(bias + d, b);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) v[j + k] = bias ? v[j + k] * inv * g[k] + b[k] : v[j + k] * inv * g[k];
+    } else {
+      v[j] = v[j] * inv * gain_vec[d];
+      if (bias) v[j] += bias[d];
+    }
   }
 }
 
-template <typename T, int NPER>
-__global__ void normed_add_norm_kernel(float* residual, const T* delta, int post_mode, const float* post_gain, float post_eps,
-                                       int out_mode, const float* gain, float eps, T* out, const int* rows, int dim,
-                                       int residual_rows) {
+template <typename T, int NPER, int VEC>
+__global__ void normed_add_norm_kernel(float* residual, NormParts parts, int post_mode, const float* post_gain, float post_eps,
+                                       int out_mode, const float* gain, const float* bias, float eps, T* out, const int* rows,
+                                       int dim, int residual_rows) {
   __shared__ float scratch[33];
   pdl_launch_dependents();
   pdl_wait();
@@ -450,55 +525,87 @@ __global__ void normed_add_norm_kernel(float* residual, const T* delta, int post
   if (!FMS_IN(src, residual_rows)) return;  // the whole block alike
   float* res = residual + (size_t)src * dim;
   float x[NPER];
-  if (delta) {
-    const T* del = delta + (size_t)src * dim;
-    float v[NPER];
 #pragma unroll
-    for (int j = 0; j < NPER; ++j) {
-      const int d = threadIdx.x + j * blockDim.x;
-      v[j] = d < dim ? to_f32(del[d]) : 0.f;
+  for (int j = 0; j < NPER; ++j) x[j] = 0.f;
+  bool changed = false;
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    if (!parts.d[k]) continue;
+    changed = true;
+    const T* del = (const T*)parts.d[k] + (size_t)src * dim;
+    const float f = k == 0 && post_mode ? 1.f : parts.s[k];
+#pragma unroll
+    for (int j = 0; j < NPER; j += VEC) {
+      const int d = (threadIdx.x + (j / VEC) * blockDim.x) * VEC;
+      if (d >= dim) continue;
+      if constexpr (VEC == 4) {
+        float v[4];
+        ldv4(del + d, v);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) x[j + e] = fmaf(f, v[e], x[j + e]);
+      } else {
+        x[j] = fmaf(f, to_f32(del[d]), x[j]);
+      }
     }
-    norm_in_registers<NPER>(v, post_mode, post_gain, post_eps, dim, scratch);
+    if (k == 0) norm_in_registers<NPER, VEC>(x, post_mode, post_gain, nullptr, post_eps, dim, scratch);
+  }
 #pragma unroll
-    for (int j = 0; j < NPER; ++j) {
-      const int d = threadIdx.x + j * blockDim.x;
-      x[j] = d < dim ? res[d] + v[j] : 0.f;
-      if (d < dim && rows == nullptr) res[d] = x[j];
-    }
-  } else {
+  for (int j = 0; j < NPER; j += VEC) {
+    const int d = (threadIdx.x + (j / VEC) * blockDim.x) * VEC;
+    if (d >= dim) continue;
+    if constexpr (VEC == 4) {
+      float v[4];
+      ldv4(res + d, v);
 #pragma unroll
-    for (int j = 0; j < NPER; ++j) {
-      const int d = threadIdx.x + j * blockDim.x;
-      x[j] = d < dim ? res[d] : 0.f;
+      for (int e = 0; e < 4; ++e) x[j + e] += v[e], v[e] = x[j + e];
+      if (changed && rows == nullptr) stv4(res + d, v);
+    } else {
+      x[j] += res[d];
+      if (changed && rows == nullptr) res[d] = x[j];
     }
   }
   if (out == nullptr) return;
-  norm_in_registers<NPER>(x, out_mode, gain, eps, dim, scratch);
+  norm_in_registers<NPER, VEC>(x, out_mode, gain, bias, eps, dim, scratch);
   T* o = out + (size_t)r * dim;
 #pragma unroll
-  for (int j = 0; j < NPER; ++j) {
-    const int d = threadIdx.x + j * blockDim.x;
-    if (d < dim) o[d] = from_f32<T>(x[j]);
+  for (int j = 0; j < NPER; j += VEC) {
+    const int d = (threadIdx.x + (j / VEC) * blockDim.x) * VEC;
+    if (d >= dim) continue;
+    if constexpr (VEC == 4) {
+      const float v[4] = {x[j], x[j + 1], x[j + 2], x[j + 3]};
+      stv4(o + d, v);
+    } else {
+      o[d] = from_f32<T>(x[j]);
+    }
   }
 }
 
-FMS_API int fms_normed_add_norm(float* residual, const void* delta, int post_mode, const float* post_gain, float post_eps,
-                                int out_mode, const float* gain, float eps, void* out, int dtype, const int* rows,
+// d0 .. d3: the parts (null: not given); post_mode != 0 norms d0 on its way (its factor is then not looked at)
+FMS_API int fms_normed_add_norm(float* residual, const void* d0, float s0, const void* d1, float s1, const void* d2, float s2,
+                                const void* d3, float s3, int post_mode, const float* post_gain, float post_eps, int out_mode,
+                                const float* gain, const float* bias, float eps, void* out, int dtype, const int* rows,
                                 int n_rows, int dim, int residual_rows, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
   if (dim <= 0 || dim > 16384) return fms_fail("normed_add_norm: rows of %d values (up to 16384)", dim);
   if (post_mode < 0 || post_mode > 2 || out_mode < 0 || out_mode > 2) return fms_fail("normed_add_norm: modes %d, %d", post_mode, out_mode);
-  if ((post_mode && delta && !post_gain) || (out_mode && out && !gain)) return fms_fail("normed_add_norm: a norm without its gain");
-  const int threads = dim >= 4096 ? 1024 : (dim >= 2048 ? 512 : (dim >= 512 ? 256 : 128));
+  if ((post_mode && d0 && !post_gain) || (out_mode && out && !gain)) return fms_fail("normed_add_norm: a norm without its gain");
+  const NormParts parts{{d0, d1, d2, d3}, {s0, s1, s2, s3}};
+  const size_t item = dtype == FMS_BF16 ? 2 : 4;
+  bool four = dim % 4 == 0 && (uintptr_t)residual % 16 == 0 && (uintptr_t)out % (4 * item) == 0 && (uintptr_t)gain % 16 == 0 &&
+              (uintptr_t)post_gain % 16 == 0 && (uintptr_t)bias % 16 == 0;
+  for (int k = 0; k < 4; ++k) four = four && (uintptr_t)parts.d[k] % (4 * item) == 0;
+  const int threads = dim >= 8192 ? 1024 : (dim >= 2048 ? 512 : (dim >= 1024 ? 256 : 128));
   const int nper = (dim + threads - 1) / threads;
-#define FMS_NAN(NPER)                                                                                                     \
-  FMS_DISPATCH_DTYPE(dtype, T, fms_launch(normed_add_norm_kernel<T, NPER>, dim3(n_rows), dim3(threads), 0, stream, residual,   \
-                                          (const T*)delta, post_mode, post_gain, post_eps, out_mode, gain, eps, (T*)out, rows, \
-                                          dim, residual_rows))
-  if (nper <= 2) FMS_NAN(2);
-  else if (nper <= 4) FMS_NAN(4);
-  else if (nper <= 8) FMS_NAN(8);
-  else FMS_NAN(16);
+#define FMS_NAN(NPER, VEC)                                                                                                  \
+  FMS_DISPATCH_DTYPE(dtype, T, fms_launch(normed_add_norm_kernel<T, NPER, VEC>, dim3(n_rows), dim3(threads), 0, stream,     \
+                                          residual, parts, post_mode, post_gain, post_eps, out_mode, gain, bias, eps, (T*)out, \
+                                          rows, dim, residual_rows))
+  if (four && nper <= 4) FMS_NAN(4, 4);
+  else if (four && nper <= 8) FMS_NAN(8, 4);
+  else if (four) FMS_NAN(16, 4);
+  else if (nper <= 4) FMS_NAN(4, 1);
+  else if (nper <= 8) FMS_NAN(8, 1);
+  else FMS_NAN(16, 1);
 #undef FMS_NAN
   return fms_launch_status("normed_add_norm");
 }
@@ -511,6 +618,7 @@ __device__ __forceinline__ float activate(float g, int act) {
     case 0: return g / (1.f + expf(-g));                                               // silu
     case 1: return 0.5f * g * (1.f + erff(g * 0.70710678118654752f));                  // gelu
     case 2: return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));  // gelu-tanh
+    case 4: g = fmaxf(g, 0.f); return g * g;                                           // the square of relu
     default: return fmaxf(g, 0.f);                                                     // relu
   }
 }
@@ -569,6 +677,98 @@ FMS_API int fms_gated_activation(const void* gu, void* out, int dtype, int n_row
                      gated_activation_kernel<T><<<blocks, threads, 0, stream>>>((const T*)gu, (T*)out, hidden, act,
                                                                                 total));
   return fms_launch_status("gated_activation");
+}
+
+// ---------------------------------------------------------------------------------------------------
+// token gate: out[t, d] = act(z[t, d]) * table[tokens[t], d]: a token's own row of a table, gated by the stream
+// ---------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void token_gate_kernel(const T* z, const T* table, const int* tokens, T* out, int dim, int vocab, int act, size_t total) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= total) return;
+  const size_t t = i / dim;
+  const int d = (int)(i - t * dim), tok = __ldcg(tokens + t);
+  const float e = tok >= 0 && tok < vocab ? to_f32(table[(size_t)tok * dim + d]) : 0.f;  // the embedding has set the flag
+  out[i] = from_f32<T>(activate(to_f32(z[i]), act) * e);
+}
+
+FMS_API int fms_token_gate(const void* z, int dtype, const void* table, const int* tokens, void* out, int n_tokens, int dim,
+                           int vocab, int act, cudaStream_t stream) {
+  if (n_tokens <= 0) return 0;
+  if (dim <= 0 || vocab <= 0 || act < 0 || act > 4) return fms_fail("token_gate: dim %d, vocab %d, activation %d", dim, vocab, act);
+  const size_t total = (size_t)n_tokens * dim;
+  FMS_DISPATCH_DTYPE(dtype, T, fms_launch(token_gate_kernel<T>, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream,
+                                          (const T*)z, (const T*)table, tokens, (T*)out, dim, vocab, act, total));
+  return fms_launch_status("token_gate");
+}
+
+// ---------------------------------------------------------------------------------------------------
+// What lies between the one projection and the one output product of a layer whose mixer and feed-forward read the same
+// input: rows [heads' results | feed-forward's hidden values] for the output matrix [Wo | Wdown].
+//   out[t, h * vdim + e]      = o[t, h * pad + e] * sigmoid(proj[t, gate_col + h * vdim + e])      (gate_col < 0: no gate)
+//   out[t, nheads * vdim + f] = act(proj[t, ff_col + f])                                           ff_gated 0
+//                             = act(proj[t, ff_col + f]) * proj[t, ff_col + hidden + f]            ff_gated 1
+// VEC values a thread (4 where sizes and addresses allow accesses of 4 values, else 1)
+// ---------------------------------------------------------------------------------------------------
+template <typename T, int VEC>
+__global__ void joint_activation_kernel(const T* o, const T* proj, int stride, int gate_col, int ff_col, T* out, int nheads,
+                                        int vdim, int pad, int hidden, int act, int ff_gated, size_t total) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+  if (i >= total) return;
+  const int heads_w = nheads * vdim, width = heads_w + hidden;
+  const size_t t = i / width;
+  const int c = (int)(i - t * width);
+  const T* row = proj + t * stride;
+  float v[VEC], g[VEC];
+  auto load = [](const T* p, float (&x)[VEC]) {
+    if constexpr (VEC == 4) ldv4(p, x);
+    else x[0] = to_f32(*p);
+  };
+  if (c < heads_w) {
+    const int h = c / vdim, e = c - h * vdim;
+    load(o + (t * nheads + h) * pad + e, v);
+    if (gate_col >= 0) {
+      load(row + gate_col + c, g);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) v[k] *= 1.f / (1.f + expf(-g[k]));
+    }
+  } else {
+    load(row + ff_col + (c - heads_w), v);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) v[k] = activate(v[k], act);
+    if (ff_gated) {
+      load(row + ff_col + hidden + (c - heads_w), g);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) v[k] *= g[k];
+    }
+  }
+  if constexpr (VEC == 4) stv4(out + i, v);
+  else out[i] = from_f32<T>(v[0]);
+}
+
+FMS_API int fms_joint_activation(const void* o, const void* proj, int stride, int gate_col, int ff_col, void* out, int dtype,
+                                 int n_tokens, int nheads, int vdim, int pad, int hidden, int act, int ff_gated,
+                                 cudaStream_t stream) {
+  if (n_tokens <= 0) return 0;
+  if (nheads <= 0 || vdim <= 0 || pad < vdim || hidden < 0 || act < 0 || act > 4)
+    return fms_fail("joint_activation: %d heads of %d (%d), %d hidden values, activation %d", nheads, vdim, pad, hidden, act);
+  const size_t total = (size_t)n_tokens * (nheads * vdim + hidden);
+  const size_t item = dtype == FMS_BF16 ? 2 : 4;
+  const bool four = vdim % 4 == 0 && pad % 4 == 0 && hidden % 4 == 0 && stride % 4 == 0 && (gate_col < 0 || gate_col % 4 == 0) &&
+                    (hidden == 0 || ff_col % 4 == 0) && (uintptr_t)o % (4 * item) == 0 && (uintptr_t)out % (4 * item) == 0 &&
+                    (uintptr_t)proj % (4 * item) == 0;
+#define FMS_JOINT(VEC)                                                                                                       \
+  FMS_DISPATCH_DTYPE(dtype, T, fms_launch(joint_activation_kernel<T, VEC>, dim3((unsigned)((total / VEC + 255) / 256)), dim3(256), \
+                                          0, stream, (const T*)o, (const T*)proj, stride, gate_col, ff_col, (T*)out, nheads, vdim, \
+                                          pad, hidden, act, ff_gated, total))
+  if (four) FMS_JOINT(4);
+  else FMS_JOINT(1);
+#undef FMS_JOINT
+  return fms_launch_status("joint_activation");
 }
 
 // ---------------------------------------------------------------------------------------------------
@@ -830,27 +1030,6 @@ FMS_API int fms_scaled_add_rmsnorm(float* residual, float alpha, const void* da,
   return fms_launch_status("scaled_add_rmsnorm");
 }
 
-// four consecutive values at once (the pointer aligned to four values)
-__device__ __forceinline__ void ldv4(const float* p, float (&v)[4]) {
-  const float4 t = *reinterpret_cast<const float4*>(p);
-  v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
-}
-__device__ __forceinline__ void ldv4(const __nv_bfloat16* p, float (&v)[4]) {
-  const uint2 t = *reinterpret_cast<const uint2*>(p);
-  v[0] = __uint_as_float(t.x << 16); v[1] = __uint_as_float(t.x & 0xffff0000u);
-  v[2] = __uint_as_float(t.y << 16); v[3] = __uint_as_float(t.y & 0xffff0000u);
-}
-__device__ __forceinline__ void stv4(float* p, const float (&v)[4]) {
-  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-}
-__device__ __forceinline__ void stv4(__nv_bfloat16* p, const float (&v)[4]) {
-  const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
-  uint2 t;
-  t.x = *reinterpret_cast<const uint32_t*>(&a);
-  t.y = *reinterpret_cast<const uint32_t*>(&b);
-  *reinterpret_cast<uint2*>(p) = t;
-}
-
 // float32 rows in the compute dtype (the stream as a sublayer's input where nothing else has made that copy)
 template <typename T>
 __global__ void cast_rows_kernel(const float* x, T* out, size_t n) {
@@ -883,11 +1062,6 @@ FMS_API int fms_cast_rows(const float* x, void* out, int dtype, long n, cudaStre
 // A warp per (row, run), or a block per (row, run) for runs of 1,024 values and more; four values a thread where the
 // run's size and the addresses allow.  The sums of a run are taken in the same order whatever else the step holds.
 // ---------------------------------------------------------------------------------------------------
-struct NormParts {
-  const void* d[4];
-  float s[4];
-};
-
 template <typename T, int VEC, bool WHOLE_BLOCK>
 __global__ void parts_group_rmsnorm_kernel(float* residual, NormParts parts, const float* gain1, const float* gain2, float eps,
                                            int groups, T* out1, T* out2, const int* rows, int n_rows, int dim, int n_res) {
@@ -1001,6 +1175,9 @@ FMS_API int fms_parts_group_rmsnorm(float* residual, const void* d0, float s0, c
 //   q, k: x / sqrt(mean(x^2) + eps) over the head's dim values, where qk_norm is set (no gain)
 //         (`norm_first`: the norm comes before the rotation, times q_gain / k_gain [dim] where those are given)
 //   `v_from_k`: there are no value columns; the value is the key as projected, before norm and rotation
+//   `v_first`: value c of a token becomes (1 - v_mix) v + v_mix v_first[t, c], mixed in float32 (the values of an
+//         earlier layer, columns of another matrix with row stride first_stride)
+//   q_out null: the queries stay where they are (heads that need nothing done are read from the projection itself)
 //   q -> q_out[t, head, 0..pad) ; k, v -> the cache row of the token's slot and place, each `pad` wide:
 //   values beyond dim (vdim) are zeros, so that kernels built for one head size `pad` serve both
 // A warp per (token, head), four a block; float32 arithmetic.
@@ -1014,7 +1191,7 @@ __global__ void qk_prepare_store_kernel(const T* proj, int stride, T* q_out, con
                                         const int* token_seq, const int* slots, T* k_cache, T* v_cache, const int* table,
                                         int table_stride, int block_tokens, int nheads, int kvheads, int dim, int vdim,
                                         int pad, int write_cache, int* error_flag, int n_seqs, int table_rows,
-                                        int pool_blocks) {
+                                        int pool_blocks, const T* v_first, int first_stride, float v_mix, int vec) {
   __shared__ float2 sc[PREP_MAX_PAIRS];
   pdl_launch_dependents();
   pdl_wait();
@@ -1028,7 +1205,7 @@ __global__ void qk_prepare_store_kernel(const T* proj, int stride, T* q_out, con
   }
   __syncthreads();
   const int lane = threadIdx.x & 31;
-  const int item = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);  // a warp per head
+  const int item = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5) + (q_out ? 0 : nheads);  // a warp per head
   const T* row = proj + (size_t)t * stride;
   T* krow = nullptr;
   T* vrow = nullptr;
@@ -1054,7 +1231,28 @@ __global__ void qk_prepare_store_kernel(const T* proj, int stride, T* q_out, con
       if (vrow == nullptr) return;
       const T* src = v_from_k ? row + (size_t)(nheads + h) * dim : row + (size_t)(nheads + kvheads) * dim + (size_t)h * vdim;
       T* dst = vrow + (size_t)h * block_tokens * pad;
-      for (int e = lane; e < pad; e += 32) dst[e] = e < vdim ? src[e] : from_f32<T>(0.f);
+      const T* first = v_first ? v_first + (size_t)t * first_stride + (size_t)h * vdim : nullptr;
+      if (vec) {
+        for (int e = 4 * lane; e < pad; e += 128) {
+          float x[4] = {0.f, 0.f, 0.f, 0.f};
+          if (e < vdim) {
+            ldv4(src + e, x);
+            if (first) {
+              float f[4];
+              ldv4(first + e, f);
+#pragma unroll
+              for (int k = 0; k < 4; ++k) x[k] = (1.f - v_mix) * x[k] + v_mix * f[k];
+            }
+          }
+          stv4(dst + e, x);
+        }
+        return;
+      }
+      for (int e = lane; e < pad; e += 32) {
+        float x = e < vdim ? to_f32(src[e]) : 0.f;
+        if (first && e < vdim) x = (1.f - v_mix) * x + v_mix * to_f32(first[e]);
+        dst[e] = from_f32<T>(x);
+      }
       return;
     }
     const bool is_q = item < nheads;
@@ -1063,6 +1261,14 @@ __global__ void qk_prepare_store_kernel(const T* proj, int stride, T* q_out, con
                   : (krow ? krow + (size_t)(item - nheads) * block_tokens * pad : nullptr);
     if (dst == nullptr) return;
     const int half = rot / 2;
+    if (vec && rot == 0 && !qk_norm) {  // nothing but the padding
+      for (int e = 4 * lane; e < pad; e += 128) {
+        float x[4] = {0.f, 0.f, 0.f, 0.f};
+        if (e < dim) ldv4(src + e, x);
+        stv4(dst + e, x);
+      }
+      return;
+    }
     if (norm_first) {
       // the norm (with its gain, where there is one) comes first and the rotation turns the normed values
       const float* gain = is_q ? q_gain : k_gain;
@@ -1110,20 +1316,27 @@ FMS_API int fms_qk_prepare_store(const void* proj, int dtype, int stride, void* 
                                  const int* token_seq, const int* slots, void* k_cache, void* v_cache, const int* table,
                                  int table_stride, int block_tokens, int n_tokens, int nheads, int kvheads, int dim,
                                  int vdim, int pad, int write_cache, int* error_flag, int n_seqs, int table_rows,
-                                 int pool_blocks, cudaStream_t stream) {
+                                 int pool_blocks, const void* v_first, int first_stride, float v_mix, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
+  if (v_first && v_from_k) return fms_fail("qk_prepare_store: values that are the keys are not mixed with others");
   if (rot < 0 || rot % 2 || rot > dim || rot / 2 > PREP_MAX_PAIRS || (rot > 0 && inv_freq == nullptr))
     return fms_fail("qk_prepare_store: %d rotated values of %d", rot, dim);
   if (dim <= 0 || vdim <= 0 || pad < dim || pad < vdim) return fms_fail("qk_prepare_store: dim %d, vdim %d, pad %d", dim, vdim, pad);
   if (v_from_k && vdim != dim) return fms_fail("qk_prepare_store: values that are the keys have the keys' size, not %d for %d", vdim, dim);
   if ((q_gain || k_gain) && !norm_first) return fms_fail("qk_prepare_store: gains belong to the norm that comes before the rotation");
+  const size_t item = dtype == FMS_BF16 ? 2 : 4;
+  const int vec = dim % 4 == 0 && vdim % 4 == 0 && pad % 4 == 0 && stride % 4 == 0 && first_stride % 4 == 0 &&
+                  (uintptr_t)proj % (4 * item) == 0 && (uintptr_t)q_out % (4 * item) == 0 && (uintptr_t)k_cache % (4 * item) == 0 &&
+                  (uintptr_t)v_cache % (4 * item) == 0 && (uintptr_t)v_first % (4 * item) == 0;
+  const int items = (q_out ? nheads : 0) + 2 * kvheads;
   FMS_DISPATCH_DTYPE(dtype, T,
-                     fms_launch(qk_prepare_store_kernel<T>, dim3(n_tokens, (nheads + 2 * kvheads + 3) / 4), dim3(128), 0, stream,
+                     fms_launch(qk_prepare_store_kernel<T>, dim3(n_tokens, (items + 3) / 4), dim3(128), 0, stream,
                                 (const T*)proj, stride,
                                 (T*)q_out, inv_freq, rot, rot_mult, qk_norm, eps, q_gain, k_gain, norm_first, halves, v_from_k,
                                 positions, position_ids, token_seq, slots,
                                 (T*)k_cache, (T*)v_cache, table, table_stride, block_tokens, nheads, kvheads, dim, vdim, pad,
-                                write_cache, error_flag, n_seqs, table_rows, pool_blocks));
+                                write_cache, error_flag, n_seqs, table_rows, pool_blocks, (const T*)v_first, first_stride, v_mix,
+                                vec));
   return fms_launch_status("qk_prepare_store");
 }
 

@@ -5,12 +5,12 @@
 //             so a step needs no answer from the device before it launches), or
 //   uniform — the same `rows` rows for every group, group g reading x at column g * x_group_offset and writing y at
 //             column g * y_group_offset (the heads of one token matrix, each with a matrix of its own).
-// With glu != 0, w[g] holds 2 N rows, [gate; up], and y = act(gate) * (up + 1) with gate cut off above `limit`, up
+// With a gated unit, w[g] holds 2 N rows, [gate; up], and y = act(gate) * (up + 1) with gate cut off above `limit`, up
 // clamped to +-limit and act(v) = v * sigmoid(alpha v): the gated unit of the routed experts.
 // Sums are float32, each output element one chain over k in order, whatever else is in the launch.
 //
 // routing: scores = sigmoid(x . router^T) in float32; the `top` largest (the lower index among equals) are a token's
-// experts and their scores its weights.  A (token, choice) pair becomes a row of the expert-sorted matrix:
+// experts and their scores its weights (further modes: fms_route).  A (token, choice) pair becomes a row of the expert-sorted matrix:
 // xs[row] = weight * x[token], rounded to the compute dtype.  After the experts, out[token] = the sum of its
 // pairs' rows in the order of its choices, float32.
 #include "common.cuh"
@@ -36,7 +36,9 @@ __device__ __forceinline__ float activated(float v, int act) {
   return v;
 }
 
-__device__ __forceinline__ float glu_clamped(float g, float u, float limit, float alpha) {
+// the gated units: act 3 is silu(gate) * up, anything else the clamped one
+__device__ __forceinline__ float glu_clamped(float g, float u, float limit, float alpha, int act = 0) {
+  if (act == 3) return g / (1.f + expf(-g)) * u;
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
   return g * (1.f / (1.f + expf(-alpha * g))) * (u + 1.f);
@@ -124,7 +126,7 @@ __global__ void __launch_bounds__(256) grouped_gemm_kernel(const T* __restrict__
     for (int j = 0; j < TN; ++j) {
       const int gn = n0 + tn + j;
       if (gn >= N) continue;
-      const float v = GLU ? glu_clamped(acc[0][i][j], acc[GLU ? 1 : 0][i][j], limit, alpha) : activated(acc[0][i][j], act);
+      const float v = GLU ? glu_clamped(acc[0][i][j], acc[GLU ? 1 : 0][i][j], limit, alpha, act) : activated(acc[0][i][j], act);
       y[(size_t)gm * y_row_stride + gn] = from_f32<T>(v);
     }
   }
@@ -245,7 +247,7 @@ __global__ void __launch_bounds__(256) grouped_rows_kernel(const T* x, const T* 
     for (int i = 0; i < 4; ++i)
       if (i < nr) {
         const float s0 = warp_sum(a0[i]), s1 = GLU ? warp_sum(a1[i]) : 0.f;
-        if (lane == 0) y[(size_t)(r0 + i) * y_row_stride + n] = from_f32<T>(GLU ? glu_clamped(s0, s1, limit, alpha) : activated(s0, act));
+        if (lane == 0) y[(size_t)(r0 + i) * y_row_stride + n] = from_f32<T>(GLU ? glu_clamped(s0, s1, limit, alpha, act) : activated(s0, act));
       }
   }
 }
@@ -294,8 +296,9 @@ template <typename T, typename TW>
 __global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(const T* __restrict__ x, const TW* __restrict__ router,
                                                     int* __restrict__ expert, float* __restrict__ weight,
                                                     int dim, int experts, int top, int mode,
-                                                    const float* __restrict__ correction, float route_scale) {
-  extern __shared__ float sm[];  // dim values of x, then `experts` logits, then (mode 1) `experts` scores
+                                                    const float* __restrict__ correction, float route_scale, int groups,
+                                                    int keep) {
+  extern __shared__ float sm[];  // dim values of x, `experts` logits, `experts` scores (mode 1, 2), `groups` scores (mode 2)
   float* xs = sm;
   float* logit = sm + dim;
   float* score = logit + experts;
@@ -336,6 +339,43 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(const T* __rest
     }
     __syncwarp();
   }
+  if (mode == 2) {
+    // scores = sigmoid(logit); the choice is by score + correction, among the experts of the best groups only
+    for (int e = lane; e < experts; e += 32) {
+      const float sc = 1.f / (1.f + expf(-logit[e]));
+      score[e] = sc;
+      logit[e] = sc + (correction ? correction[e] : 0.f);
+    }
+    __syncwarp();
+    if (keep < groups) {
+      // a group of neighbours scores the sum of its two largest choice scores; the `keep` best groups stay (the lower
+      // index among equals), the other groups' experts cannot be chosen
+      float* group_score = score + experts;
+      const int size = experts / groups;
+      for (int g = lane; g < groups; g += 32) {
+        float first = -INFINITY, second = -INFINITY;
+        for (int e = g * size; e < (g + 1) * size; ++e) {
+          const float v = logit[e];
+          if (v > first) {
+            second = first;
+            first = v;
+          } else if (v > second) {
+            second = v;
+          }
+        }
+        group_score[g] = size > 1 ? first + second : first;
+      }
+      __syncwarp();
+      for (int e = lane; e < experts; e += 32) {
+        const int mine = e / size;
+        const float v = group_score[mine];
+        int better = 0;
+        for (int g = 0; g < groups; ++g) better += group_score[g] > v || (group_score[g] == v && g < mine) ? 1 : 0;
+        if (better >= keep) logit[e] = -INFINITY;
+      }
+      __syncwarp();
+    }
+  }
   float picked_sum = 0.f;
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
@@ -359,7 +399,7 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(const T* __rest
     if (at >= experts) at = k;  // every logit was NaN or -inf: any expert, so that nothing below reads outside
     if (lane == 0) {
       expert[(size_t)t * top + k] = at;
-      weight[(size_t)t * top + k] = mode == 1 ? score[at] : 1.f / (1.f + expf(-best));
+      weight[(size_t)t * top + k] = mode == 1 ? score[at] : (mode == 2 ? score[at] * route_scale : 1.f / (1.f + expf(-best)));
       logit[at] = -INFINITY;
     }
     if (mode == 1) picked_sum += score[at];
@@ -460,15 +500,16 @@ FMS_API int fms_grouped_tile_rows() { return BM; }
 
 // offsets null: uniform groups of `rows` rows; else ragged groups, `rows` = all rows of x, and tile_first as
 // fms_route leaves it.  few_rows != 0: the kernel that walks each group's rows (a decode step).
-// glu: 0 plain, 1 the gated unit over [gate; up] rows, 2 an ungated product whose sums are squared where positive.
+// glu: 0 plain, 1 the clamped gated unit over [gate; up] rows, 2 an ungated product whose sums are squared where
+// positive, 3 silu(gate) * up over [gate; up] rows.
 FMS_API int fms_grouped_linear(const void* x, const void* w, void* y, int dtype, const int* offsets, const int* tile_first,
                                const int* group_of_row, int groups, int rows, int N, int K, long x_row_stride,
                                long x_group_offset, long y_row_stride, long y_group_offset, int glu, float limit,
                                float alpha, int few_rows, cudaStream_t stream) {
   if (rows <= 0 || groups <= 0 || N <= 0) return 0;
   if (K <= 0) return fms_fail("grouped_linear: K %d", K);
-  const int act = glu == 2 ? 2 : 0;
-  glu = glu == 1 ? 1 : 0;
+  const int act = glu == 2 ? 2 : (glu == 3 ? 3 : 0);
+  glu = glu == 1 || glu == 3 ? 1 : 0;
   if (few_rows) {
     if (groups > 65535) return fms_fail("grouped_linear: %d groups are more than the row-by-row kernel takes", groups);
     dim3 grid((N + 7) / 8, groups);
@@ -509,19 +550,24 @@ FMS_API int fms_grouped_linear(const void* x, const void* w, void* y, int dtype,
 // counts [experts] is scratch: the rows of each expert that are placed so far.
 // mode 0: scores sigmoid(logit), the rows of xs are the tokens' times their weights.  mode 1: scores softmax(logits), the
 // choice by score + correction [experts] (float32 or null), weights the chosen scores over their sum times route_scale;
-// the rows of xs are the tokens' as they are and fms_route_gather takes the weights.
+// the rows of xs are the tokens' as they are and fms_route_gather takes the weights.  mode 2: scores sigmoid(logit), the
+// choice by score + correction among the experts of the `keep` best of `groups` equal groups of neighbours (a group's
+// score: the sum of its two largest choice scores), weights the chosen scores times route_scale; rows as in mode 1.
 FMS_API int fms_route(const void* x, int dtype, const void* router, int router_dtype, int* expert, float* weight, int* counts,
                       int* offsets, int* tile_first, int* row_of_pair, int* group_of_row, void* xs, int n_tokens, int dim,
-                      int experts, int top, int mode, const float* correction, float route_scale, cudaStream_t stream) {
+                      int experts, int top, int mode, const float* correction, float route_scale, int groups, int keep,
+                      cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (dim <= 0 || experts <= 0 || top <= 0 || top > experts) return fms_fail("route: dim %d, experts %d, top %d", dim, experts, top);
-  if (mode != 0 && mode != 1) return fms_fail("route: mode %d", mode);
-  const size_t smem = ((size_t)dim + 2 * (size_t)experts) * sizeof(float);
+  if (mode < 0 || mode > 2) return fms_fail("route: mode %d", mode);
+  if (groups <= 0 || experts % groups || keep <= 0 || keep > groups || (long)keep * (experts / groups) < top)
+    return fms_fail("route: %d experts in %d groups of which %d stay, top %d", experts, groups, keep, top);
+  const size_t smem = ((size_t)dim + 2 * (size_t)experts + (size_t)groups) * sizeof(float);
   if (smem > 200 * 1024) return fms_fail("route: rows of %d values and %d experts do not fit shared memory", dim, experts);
   FMS_DISPATCH_DTYPE(dtype, T, FMS_DISPATCH_DTYPE(router_dtype, TW, {
     if (smem > 48 * 1024) cudaFuncSetAttribute(route_kernel<T, TW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     fms_launch(route_kernel<T, TW>, dim3(n_tokens), dim3(32 * ROUTE_WARPS), smem, stream, (const T*)x, (const TW*)router, expert, weight,
-               dim, experts, top, mode, correction, route_scale);
+               dim, experts, top, mode, correction, route_scale, groups, keep);
   }));
   if (fms_launch_status("route")) return 1;
   const int n_pairs = n_tokens * top;

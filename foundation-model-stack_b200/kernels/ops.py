@@ -34,6 +34,9 @@ _P, _I, _F, _U64, _L = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_u
 
 _SIGNATURES = {
     "fms_embed_rows": [_P, _I, _P, _P, _I, _I, _I, _F, _P, _P],
+    "fms_embed_rows_at": [_P, _I, _P, _P, _I, _I, _I, _F, _P, _P, _I, _P, _P],
+    "fms_token_gate": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _P],
+    "fms_joint_activation": [_P, _P, _I, _I, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     "fms_add_rmsnorm": [_P, _P, _P, _I, _F, _P, _I, _P, _I, _I, _I, _P],
     "fms_gated_activation": [_P, _P, _I, _I, _I, _I, _P],
     "fms_rope_store": [_P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _I, _P],
@@ -56,7 +59,7 @@ _SIGNATURES = {
     "fms_normed_add_rmsnorm": [_P, _P, _I, _P, _F, _F, _P, _F, _F, _I, _P, _I, _P, _I, _I, _I, _P],
     "fms_mingru_scan": [_P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _P, _P, _I, _P, _P],
     "fms_grouped_linear": [_P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _L, _L, _L, _L, _I, _F, _F, _I, _P],
-    "fms_route": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _F, _P],
+    "fms_route": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _F, _I, _I, _P],
     "fms_route_gather": [_P, _I, _P, _P, _I, _I, _I, _P, _P],
     "fms_relu_squared": [_P, _I, _L, _P],
     "fms_gated_clamped": [_P, _P, _I, _I, _I, _F, _F, _P],
@@ -71,17 +74,17 @@ _SIGNATURES = {
     "fms_cast_rows": [_P, _P, _I, _L, _P],
     "fms_parts_group_rmsnorm": [_P, _P, _F, _P, _F, _P, _F, _P, _F, _P, _P, _F, _I, _P, _P, _I, _P, _I, _I, _I, _P],
     "fms_qk_prepare_store": [_P, _I, _I, _P, _P, _I, _F, _I, _F, _P, _P, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I,
-                             _I, _I, _I, _I, _I, _P, _I, _I, _I, _P],
+                             _I, _I, _I, _I, _I, _P, _I, _I, _I, _P, _I, _F, _P],
     "fms_sigmoid_gate": [_P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _I, _P],
-    "fms_normed_add_norm": [_P, _P, _I, _P, _F, _I, _P, _F, _P, _I, _P, _I, _I, _I, _P],
+    "fms_normed_add_norm": [_P, _P, _F, _P, _F, _P, _F, _P, _F, _I, _P, _F, _I, _P, _P, _F, _P, _I, _P, _I, _I, _I, _P],
     "fms_linear_prepare": [_P, _I, _I, _P, _I, _I, _I, _F, _I, _P],
     "fms_decay_scan": [_P, _P, _I, _I, _P, _F, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "fms_attention_prefill_sink": [_P, _P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P,
                                    _P],
     "fms_attention_prefill_masked": [_P, _P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P,
-                                     _I, _F, _P],
+                                     _I, _F, _P, _L, _P],
     "fms_attention_decode_masked": [_P, _P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _F, _I, _I, _I, _L,
-                                    _P, _P, _P, _I, _F, _P],
+                                    _P, _P, _P, _I, _F, _P, _L, _P],
     "fms_attention_decode_sink": [_P, _P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _F, _I, _I, _I, _L,
                                   _P, _P, _P, _P],
     "fms_causal_conv": [_P, _I, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
@@ -199,7 +202,8 @@ def check_error_flag(device) -> None:
                            2: "a token's position has no cache block",
                            4: "a kernel gave up waiting for a copy or for the tensor cores",
                            8: "decode attention was launched with fewer key splits than a sequence's length needs",
-                           16: "a kernel's bounds check met an index outside its array"}.get(v, f"device error flag {v}"))
+                           16: "a kernel's bounds check met an index outside its array",
+                           32: "a position outside the table of learned positions reached the embedding"}.get(v, f"device error flag {v}"))
 
 
 # ---- embedding ---------------------------------------------------------------------------------------
@@ -209,6 +213,20 @@ def embed(table: torch.Tensor, tokens: torch.Tensor, scale: float = 1.0) -> torc
     out = torch.empty((n, dim), dtype=torch.float32, device=table.device)
     _call("elementwise", "fms_embed_rows", _ptr(table), _code(table.dtype), _ptr(tokens), _ptr(out), n, dim,
           table.shape[0], float(scale), _ptr(error_flag(table.device)), _stream())
+    return out
+
+
+def embed_at(table: torch.Tensor, positions_table: torch.Tensor, batch, scale: float = 1.0) -> torch.Tensor:
+    """Float32 rows ``scale`` * table[token] + positions_table[position] of a step's tokens; a row's position is
+    ``batch.position_ids`` where the batch has them, else its place in the cache."""
+    n, dim = batch.tokens.shape[0], table.shape[1]
+    if positions_table.dtype != table.dtype or positions_table.shape[1] != dim:
+        raise KernelError("embed_at: the table of positions has the token table's dtype and width")
+    ids = getattr(batch, "position_ids", None)
+    out = torch.empty((n, dim), dtype=torch.float32, device=table.device)
+    _call("elementwise", "fms_embed_rows_at", _ptr(table), _code(table.dtype), _ptr(batch.tokens), _ptr(out), n, dim,
+          table.shape[0], float(scale), _ptr(positions_table), _ptr(batch.positions if ids is None else ids),
+          positions_table.shape[0], _ptr(error_flag(table.device)), _stream())
     return out
 
 
@@ -257,27 +275,35 @@ def normed_add_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], po
 NORM_NONE, NORM_RMS, NORM_LAYER = 0, 1, 2
 
 
-def normed_add_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], post, out_norm, out_dtype: torch.dtype,
-                    rows: Optional[torch.Tensor] = None, want_out: bool = True) -> Optional[torch.Tensor]:
+def normed_add_norm(residual: torch.Tensor, delta, post, out_norm, out_dtype: torch.dtype,
+                    rows: Optional[torch.Tensor] = None, want_out: bool = True,
+                    bias: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """residual (float32, in place) += post(delta); returns out_norm(residual) in ``out_dtype``.  ``post`` and
     ``out_norm`` are (mode, gain, eps) with mode ``NORM_NONE`` (the rows as they are), ``NORM_RMS`` or ``NORM_LAYER``
-    (the mean taken off, the variance the mean of the squared deviations, no bias) and gain a float32 vector of the
-    row's width (None with ``NORM_NONE``).  With ``rows`` only those rows are computed and the residual is not written.
-    ``want_out`` False: only the sum is wanted and nothing is returned."""
+    (the mean taken off, the variance the mean of the squared deviations) and gain a float32 vector of the
+    row's width (None with ``NORM_NONE``); ``bias`` (float32, or None) is added to the result.  ``delta`` may also be a
+    list of up to four (delta, factor), whose weighted sum is added (with no ``post``).  With ``rows`` only those rows
+    are computed and the residual is not written.  ``want_out`` False: only the sum is wanted and nothing is returned."""
     dim = residual.shape[1]
     n = rows.shape[0] if rows is not None else residual.shape[0]
     if residual.dtype != torch.float32:
         raise KernelError("the residual stream is float32")
-    if delta is not None and delta.dtype != out_dtype:
-        raise KernelError(f"sublayer output is {delta.dtype}, compute dtype is {out_dtype}")
+    parts = list(delta) if isinstance(delta, (list, tuple)) else ([] if delta is None else [(delta, 1.0)])
+    if len(parts) > 4 or any(d.dtype != out_dtype or tuple(d.shape) != tuple(residual.shape) for d, _ in parts):
+        raise KernelError(f"normed_add_norm: up to four sublayer outputs of the stream's shape in the compute dtype, {out_dtype}")
     post_mode, post_gain, post_eps = post if post is not None else (NORM_NONE, None, 0.0)
+    if post_mode != NORM_NONE and len(parts) > 1:
+        raise KernelError("normed_add_norm: one output is normed on its way, not several")
     out_mode, gain, eps = out_norm if out_norm is not None else (NORM_NONE, None, 0.0)
-    for g in (post_gain, gain):
+    flat = []
+    for i in range(4):
+        flat += [_ptr(parts[i][0]), float(parts[i][1])] if i < len(parts) else [None, 0.0]
+    for g in (post_gain, gain, bias):
         if g is not None and (g.dtype != torch.float32 or g.shape[0] != dim):
             raise KernelError("normed_add_norm: gains are float32 vectors of the row's width")
     out = torch.empty((n, dim), dtype=out_dtype, device=residual.device) if want_out else None
-    _call("elementwise", "fms_normed_add_norm", _ptr(residual), _ptr(delta), int(post_mode), _ptr(post_gain), float(post_eps),
-          int(out_mode), _ptr(gain), float(eps), _ptr(out), _code(out_dtype), _ptr(rows), n, dim, residual.shape[0], _stream())
+    _call("elementwise", "fms_normed_add_norm", _ptr(residual), *flat, int(post_mode), _ptr(post_gain), float(post_eps),
+          int(out_mode), _ptr(gain), _ptr(bias), float(eps), _ptr(out), _code(out_dtype), _ptr(rows), n, dim, residual.shape[0], _stream())
     return out
 
 
@@ -490,6 +516,32 @@ def gated_activation(gate_up: torch.Tensor, activation: int) -> torch.Tensor:
     return out
 
 
+def token_gate(z: torch.Tensor, table: torch.Tensor, tokens: torch.Tensor, activation: int) -> torch.Tensor:
+    """act(z[t]) * table[tokens[t]]: rows of a table, one a token, gated by ``z`` [tokens, dim]."""
+    n, dim = z.shape
+    if table.dtype != z.dtype or table.shape[1] != dim:
+        raise KernelError(f"token_gate: z {z.dtype} {tuple(z.shape)}, table {table.dtype} {tuple(table.shape)}")
+    out = torch.empty_like(z)
+    _call("elementwise", "fms_token_gate", _ptr(z), _code(z.dtype), _ptr(table), _ptr(tokens), _ptr(out), n, dim, table.shape[0],
+          int(activation), _stream())
+    return out
+
+
+def joint_activation(o: torch.Tensor, proj: torch.Tensor, gate_col: int, ff_col: int, nheads: int, vdim: int, pad: int,
+                     hidden: int, activation: int, gated: bool) -> torch.Tensor:
+    """[tokens, nheads * vdim + hidden]: the heads' results ``o`` (heads of ``pad`` values, of which ``vdim`` count) times
+    sigmoid of ``proj``'s columns from ``gate_col`` on (negative: no gate), then the feed-forward's hidden values,
+    act(proj[:, ff_col:]) or, ``gated``, act of the first ``hidden`` columns times the next ``hidden``."""
+    n = o.shape[0]
+    if proj.dtype != o.dtype or proj.shape[0] != n or o.shape[1] != nheads * pad \
+            or proj.shape[1] < max(gate_col + nheads * vdim, ff_col + hidden * (2 if gated else 1) if hidden else 0):
+        raise KernelError(f"joint_activation: o {o.dtype} {tuple(o.shape)}, proj {proj.dtype} {tuple(proj.shape)}")
+    out = torch.empty((n, nheads * vdim + hidden), dtype=o.dtype, device=o.device)
+    _call("elementwise", "fms_joint_activation", _ptr(o), _ptr(proj), proj.shape[1], int(gate_col), int(ff_col), _ptr(out),
+          _code(o.dtype), n, nheads, vdim, pad, hidden, int(activation), 1 if gated else 0, _stream())
+    return out
+
+
 # ---- attention ---------------------------------------------------------------------------------------
 def rope_store(qkv: torch.Tensor, inv_freq: Optional[torch.Tensor], batch, view, nheads: int, kvheads: int,
                head_dim: int, writes_cache: bool = True) -> torch.Tensor:
@@ -595,29 +647,41 @@ def qk_prepare_store(proj: torch.Tensor, inv_freq: Optional[torch.Tensor], rot: 
                      view, nheads: int, kvheads: int, dim: int, vdim: int, pad: int,
                      writes_cache: bool = True, norm_first: bool = False, q_gain: Optional[torch.Tensor] = None,
                      k_gain: Optional[torch.Tensor] = None, halves: bool = False, values_are_keys: bool = False,
-                     rot_mult: float = 1.0) -> torch.Tensor:
+                     rot_mult: float = 1.0, q_in_place: bool = False, first_values=None, v_mix: float = 0.0) -> Optional[torch.Tensor]:
     """From rows [q: nheads x dim | k: kvheads x dim | v: kvheads x vdim | ...] of ``proj``: rotates the first ``rot``
     values of every q and k head by the row's position (adjacent pairs; with ``halves`` value i with value i + rot / 2),
     divides q and k by their root mean square over ``dim`` where ``qk_norm`` (after the rotation; with ``norm_first``
     before it, and then times ``q_gain`` / ``k_gain``, float32 [dim], where given), writes k and v into the cache (heads
     of ``pad`` values there, zeros beyond dim and vdim) and returns q [tokens, nheads * pad], padded alike.
     ``values_are_keys``: the rows have no v columns; a value is its key as projected, before norm and rotation.
-    ``rot_mult`` multiplies the rotation's sines and cosines (stretched frequencies come with such a constant)."""
+    ``rot_mult`` multiplies the rotation's sines and cosines (stretched frequencies come with such a constant).
+    ``q_in_place``: the queries need nothing (no rotation, no norm, no padding) and are left where they are; returns None.
+    ``first_values`` (matrix, column): the values become (1 - v_mix) v + v_mix first, mixed in float32, with first the
+    kvheads * vdim columns of that matrix from that column on."""
     n = proj.shape[0]
+    first_ptr = first_stride = None
+    if first_values is not None:
+        first, col = first_values
+        if first.dtype != proj.dtype or first.shape[0] != n or first.shape[1] < col + kvheads * vdim:
+            raise KernelError(f"qk_prepare_store: the values to mix in are {first.dtype} {tuple(first.shape)} from column {col}")
+        first_ptr, first_stride = _ptr(first) + col * first.element_size(), first.shape[1]
+    if q_in_place and (rot or qk_norm or pad != dim):
+        raise KernelError("qk_prepare_store: queries that are rotated, normed or padded are not left in place")
     for g in (q_gain, k_gain):
         if g is not None and (g.dtype != torch.float32 or g.shape[0] != dim):
             raise KernelError("qk_prepare_store: gains are float32 vectors of the head's size")
     if view.keys.dtype != proj.dtype or view.keys.shape[-1] != pad:
         raise KernelError(f"cache is {view.keys.dtype} with heads of {view.keys.shape[-1]}, activations are {proj.dtype}, "
                           f"heads of {pad}")
-    q = torch.empty((n, nheads * pad), dtype=proj.dtype, device=proj.device)
+    q = None if q_in_place else torch.empty((n, nheads * pad), dtype=proj.dtype, device=proj.device)
     _call("elementwise", "fms_qk_prepare_store", _ptr(proj), _code(proj.dtype), proj.shape[1], _ptr(q), _ptr(inv_freq),
           int(rot), float(rot_mult), 1 if qk_norm else 0, float(eps), _ptr(q_gain), _ptr(k_gain), 1 if norm_first else 0,
           1 if halves else 0,
           1 if values_are_keys else 0, _ptr(batch.positions), _ptr(getattr(batch, "position_ids", None)),
           _ptr(batch.token_seq), _ptr(batch.slots), _ptr(view.keys), _ptr(view.values), _ptr(view.table),
           view.table.shape[1], view.block_tokens, n, nheads, kvheads, dim, vdim, pad, 1 if writes_cache else 0,
-          _ptr(error_flag(proj.device)), batch.slots.shape[0], view.table.shape[0], view.keys.shape[0], _stream())
+          _ptr(error_flag(proj.device)), batch.slots.shape[0], view.table.shape[0], view.keys.shape[0], first_ptr,
+          first_stride or 0, float(v_mix), _stream())
     return q
 
 
@@ -635,19 +699,25 @@ def sigmoid_gate(o: torch.Tensor, gate: Optional[torch.Tensor], gate_offset: int
 
 
 def attention(q: torch.Tensor, batch, view, nheads: int, kvheads: int, head_dim: int, scale: float,
-              window: int, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0) -> torch.Tensor:
+              window: int, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0,
+              distance: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal softmax attention of the step's queries over the cache (which already holds the step's own
     keys and values).  One query per sequence takes the split-key decode kernels, else the prefill kernel.
     ``sink`` [nheads] float32: a term exp(sink[h]) in every row's denominator that belongs to no key.
     ``chunk`` > 0: the positions of a sequence are cut into runs of ``chunk``, counted from its position 0, and a query
     sees the keys of its own run only (not together with a window).  ``softcap`` > 0: a score s becomes
-    softcap * tanh(s / softcap) after the scale."""
-    masked = bool(chunk) or bool(softcap)
+    softcap * tanh(s / softcap) after the scale.  ``distance`` [nheads, 2] float32, pairs (r1, r2): then
+    r1 * ln(1 + r2 * (query position - key position)) is taken off the score.  The queries are the first nheads *
+    head_dim columns of ``q``, which may be wider."""
+    wide = q.shape[1] != nheads * head_dim
+    masked = bool(chunk) or bool(softcap) or distance is not None or wide
+    if distance is not None and (distance.dtype != torch.float32 or tuple(distance.shape) != (nheads, 2)):
+        raise KernelError("attention: the distance term is float32, two numbers a head")
     if chunk < 0 or softcap < 0 or (chunk and window):
         raise KernelError(f"attention: chunk {chunk}, window {window}, softcap {softcap}")
     if sink is not None and (sink.dtype != torch.float32 or sink.shape[0] != nheads):
         raise KernelError("attention: the sinks are float32, one per head")
-    out = torch.empty_like(q)
+    out = torch.empty((q.shape[0], nheads * head_dim), dtype=q.dtype, device=q.device)
     lib = _attention_library(head_dim)
     split, tile_rows = attention_constants(head_dim, q.dtype, nheads, kvheads)
     common = (_ptr(q), _ptr(out), _code(q.dtype), _ptr(view.keys), _ptr(view.values), _ptr(view.table),
@@ -657,7 +727,8 @@ def attention(q: torch.Tensor, batch, view, nheads: int, kvheads: int, head_dim:
         part_o = torch.empty((batch.n_seqs, nheads, n_splits, head_dim), dtype=torch.float32, device=q.device)
         part_ml = torch.empty((batch.n_seqs, nheads, n_splits, 2), dtype=torch.float32, device=q.device)
         # total_len (what the host knows of the sequences' lengths) chooses between the two bfloat16 decode kernels
-        tail = (_ptr(sink), int(chunk), float(softcap)) if masked else (() if sink is None else (_ptr(sink),))
+        tail = (_ptr(sink), int(chunk), float(softcap), _ptr(distance), q.shape[1]) if masked else \
+            (() if sink is None else (_ptr(sink),))
         _call(lib, "fms_attention_decode_masked" if masked else
               ("fms_attention_decode" if sink is None else "fms_attention_decode_sink"), *common, batch.n_seqs,
               n_splits, _ptr(part_o), _ptr(part_ml), nheads,
@@ -669,7 +740,8 @@ def attention(q: torch.Tensor, batch, view, nheads: int, kvheads: int, head_dim:
             launches += 1  # the kernel that merges the splits
     else:
         tiles = batch.query_tiles(tile_rows)
-        tail = (_ptr(sink), int(chunk), float(softcap)) if masked else (() if sink is None else (_ptr(sink),))
+        tail = (_ptr(sink), int(chunk), float(softcap), _ptr(distance), q.shape[1]) if masked else \
+            (() if sink is None else (_ptr(sink),))
         _call(lib, "fms_attention_prefill_masked" if masked else
               ("fms_attention_prefill" if sink is None else "fms_attention_prefill_sink"), *common, _ptr(tiles),
               tiles.shape[0], nheads, kvheads, head_dim, float(scale), int(window), view.keys.shape[0],
@@ -903,16 +975,19 @@ class Routing:
                  "weights_on_output")
 
 
-ROUTE_SIGMOID, ROUTE_SOFTMAX = 0, 1
+ROUTE_SIGMOID, ROUTE_SOFTMAX, ROUTE_SIGMOID_GROUPS = 0, 1, 2
 
 
 def route(x: torch.Tensor, router: torch.Tensor, top: int, mode: int = ROUTE_SIGMOID,
-          correction: Optional[torch.Tensor] = None, route_scale: float = 1.0) -> Routing:
+          correction: Optional[torch.Tensor] = None, route_scale: float = 1.0, groups: int = 1, keep: int = 1) -> Routing:
     """``ROUTE_SIGMOID``: scores sigmoid(x router^T) in float32; every token's ``top`` best experts; rows
     weight * x[token] sorted by expert.  ``ROUTE_SOFTMAX``: scores softmax(x router^T) over all experts; the ``top``
     experts with the largest score + ``correction`` [experts] (float32, or None) are the token's; its weights are their
     scores over their sum (+ 1e-20), times ``route_scale``; the sorted rows are the tokens' as they are and
-    ``route_gather`` multiplies the experts' results by the weights."""
+    ``route_gather`` multiplies the experts' results by the weights.  ``ROUTE_SIGMOID_GROUPS``: scores sigmoid(x
+    router^T); the choice is by score + ``correction`` among the experts of the ``keep`` best of ``groups`` equal groups of
+    neighbours (a group's score: the sum of its two largest choice scores); the weights are the chosen scores (without
+    the correction) times ``route_scale``, and multiply the results as with ``ROUTE_SOFTMAX``."""
     if correction is not None and (correction.dtype != torch.float32 or correction.shape[0] != router.shape[0]):
         raise KernelError("route: the correction is float32, one number an expert")
     n, dim = x.shape
@@ -920,7 +995,7 @@ def route(x: torch.Tensor, router: torch.Tensor, top: int, mode: int = ROUTE_SIG
     dev = x.device
     r = Routing()
     r.top, r.experts = top, experts
-    r.weights_on_output = mode == ROUTE_SOFTMAX
+    r.weights_on_output = mode != ROUTE_SIGMOID
     ints = torch.empty((n * top * 3 + 3 * (experts + 1),), dtype=torch.int32, device=dev)
     r.expert = ints[: n * top].view(n, top)
     r.row_of_pair = ints[n * top: 2 * n * top]
@@ -933,17 +1008,18 @@ def route(x: torch.Tensor, router: torch.Tensor, top: int, mode: int = ROUTE_SIG
     r.rows = torch.empty((n * top, dim), dtype=x.dtype, device=dev)
     _call("grouped", "fms_route", _ptr(x), _code(x.dtype), _ptr(router), _code(router.dtype), _ptr(r.expert),
           _ptr(r.weight), _ptr(counts), _ptr(r.offsets), _ptr(r.tile_first), _ptr(r.row_of_pair), _ptr(r.group_of_row),
-          _ptr(r.rows), n, dim, experts, top, int(mode), _ptr(correction), float(route_scale), _stream())
+          _ptr(r.rows), n, dim, experts, top, int(mode), _ptr(correction), float(route_scale), int(groups), int(keep),
+          _stream())
     global launches
     launches += 2
     return r
 
 
 def routed_linear(rows: torch.Tensor, weight: torch.Tensor, routing: Routing, glu: bool = False, limit: float = 0.0,
-                  alpha: float = 1.0, relu_squared: bool = False) -> torch.Tensor:
+                  alpha: float = 1.0, relu_squared: bool = False, silu: bool = False) -> torch.Tensor:
     """Ragged groups: y[r] = rows[r] . weight[expert of r]^T; with ``glu`` weight[e] = [gate; up] and
-    y = g * sigmoid(alpha g) * (u + 1) for g = min(gate, limit), u = clamp(up, -limit, limit); with ``relu_squared``
-    y = max(y, 0)^2."""
+    y = g * sigmoid(alpha g) * (u + 1) for g = min(gate, limit), u = clamp(up, -limit, limit), or, with ``silu`` too,
+    y = silu(gate) * up; with ``relu_squared`` y = max(y, 0)^2."""
     n, k = rows.shape
     n_out = weight.shape[1] // (2 if glu else 1)
     if weight.dtype != rows.dtype or weight.shape[0] != routing.experts or weight.shape[2] != k:
@@ -958,6 +1034,8 @@ def routed_linear(rows: torch.Tensor, weight: torch.Tensor, routing: Routing, gl
             _call("grouped", "fms_relu_squared", _ptr(y), _code(y.dtype), y.numel(), _stream())
         if not glu:
             return y
+        if silu:
+            return gated_activation(y, 0)
         out = torch.empty((n, n_out), dtype=rows.dtype, device=rows.device)
         _call("grouped", "fms_gated_clamped", _ptr(y), _ptr(out), _code(y.dtype), n, n_out, float(limit), float(alpha),
               _stream())
@@ -965,7 +1043,7 @@ def routed_linear(rows: torch.Tensor, weight: torch.Tensor, routing: Routing, gl
     y = torch.empty((n, n_out), dtype=rows.dtype, device=rows.device)
     _call("grouped", "fms_grouped_linear", _ptr(rows), _ptr(weight), _ptr(y), _code(rows.dtype), _ptr(routing.offsets),
           _ptr(routing.tile_first), _ptr(routing.group_of_row), routing.experts, n, n_out, k, k, 0, n_out, 0,
-          1 if glu else (2 if relu_squared else 0), float(limit), float(alpha), 1 if n <= GROUPED_FEW_ROWS else 0, _stream())
+          (3 if silu else 1) if glu else (2 if relu_squared else 0), float(limit), float(alpha), 1 if n <= GROUPED_FEW_ROWS else 0, _stream())
     return y
 
 

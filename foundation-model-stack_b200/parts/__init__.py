@@ -4,7 +4,7 @@ from .registry import (build_block, build_embedding, build_feed_forward, build_m
                        register_block, register_embedding, register_feed_forward, register_mixer, register_norm,
                        register_position, registered)
 from . import (norm, position, attention, feedforward, embedding, recurrent, latent_attention,  # noqa: F401  (registration)
-               experts, state_space)
+               experts, state_space, token_side)
 from .block import Block, PostNormBlock, PreNormBlock, SandwichBlock, ScaledParts
 from .norm import NormedDelta, StreamCopy
 from .linear import Linear

@@ -86,6 +86,12 @@ class SinkAttention(Part):
         keys seen in runs (``chunk`` = n: the positions of a sequence are cut into runs of n, counted from its position 0,
             and a query sees the keys of its own run up to itself; instead of a window)
         capped scores (``softcap`` = c: s becomes c * tanh(s / c) after the scale)
+        a distance term (``distance``): r1[h] * ln(1 + r2[h] * (i - j)) is taken off the score of query i and key j, after
+            the cap; tensors ``r1`` and ``r2`` [nheads]
+        values mixed with an earlier layer's (``v_mix``): "first": the layer's values are handed to the layers after it;
+            "mixed": v becomes (1 - vmix) v + vmix v_first, in float32, before it is cached, with the values of the layer
+            that said "first" for the same token and one number ``vmix`` (a tensor without dimensions; a "first" layer
+            may have one too and does not use it)
         a bias on the output projection (``out_bias``)
         frequencies stretched by a ramp ("yarn" scaling of ``position``): the sines and cosines are then also multiplied
             by the constant that belongs to it
@@ -95,7 +101,11 @@ class SinkAttention(Part):
     of ``pad`` = max(head_dim, vdim) rounded up to 16 values, zeros beyond each one's own size, so that the attention
     kernels built for one head size serve keys and values alike; q is padded the same way and the padding of the
     result is dropped by the gate kernel.  ``out_factor`` multiplies the result before the output projection (a mixer
-    that stands beside another one carries its weight there)."""
+    that stands beside another one carries its weight there).
+
+    With ``projections`` "outside" the mixer has neither projection: a block that projects for several sublayers at once
+    hands ``attend`` a matrix whose first ``in_rows`` columns are the fused projection's, and makes the output product
+    over ``out_columns`` values itself, after the gate (``gate_col``) and the padding (``pad``)."""
 
     def __init__(self, spec: MixerSpec) -> None:
         super().__init__()
@@ -134,14 +144,31 @@ class SinkAttention(Part):
         self.gate_col = (self.nheads + self.kvheads) * self.head_dim + (0 if self.values_are_keys else self.kvheads * self.vdim)
         rows = self.fused_rows(self.nheads, self.kvheads, self.head_dim, self.vdim, self.values_are_keys,
                                o.get("gate", False))
-        self.in_proj = self.add("in_proj", Linear(spec.dim, rows, spec.bias))
+        self.in_rows, self.out_columns = rows, self.nheads * self.vdim
+        self.value_col = (self.nheads + self.kvheads) * self.head_dim
+        self.projects = o.get("projections", "own") == "own"
+        if not self.projects and (self.gate_per_head or self.out_factor != 1.0 or spec.bias or o.get("out_bias", False)):
+            raise ValueError("sink_attention: projections from outside go with one gate a value, without biases and factor")
+        if self.projects:
+            self.in_proj = self.add("in_proj", Linear(spec.dim, rows, spec.bias))
+        self.has_distance = bool(o.get("distance", False))
+        if self.has_distance:
+            self.declare("r1", (self.nheads,), role="vector")
+            self.declare("r2", (self.nheads,), role="vector")
+        self.v_mix = o.get("v_mix") or ""
+        if self.v_mix not in ("", "first", "mixed") or (self.v_mix and self.values_are_keys):
+            raise ValueError(f"sink_attention: v_mix {self.v_mix!r}, values {o.get('values', 'projected')!r}")
+        if self.v_mix:
+            self.declare("vmix", (), role="vector", optional=self.v_mix == "first")
         if self.has_sink:
             self.declare("sink", (self.nheads,), role="vector")
         if self.norm_first:
             self.declare("q_norm", (self.head_dim,), role="vector")
             self.declare("k_norm", (self.head_dim,), role="vector")
-        self.dense = self.add("dense", Linear(self.nheads * self.vdim, spec.dim, bool(o.get("out_bias", False))))
-        self._inv_freq = self._sink = self._q_gain = self._k_gain = None
+        if self.projects:
+            self.dense = self.add("dense", Linear(self.nheads * self.vdim, spec.dim, bool(o.get("out_bias", False))))
+        self._inv_freq = self._sink = self._q_gain = self._k_gain = self._distance = None
+        self._mix = 0.0
 
     @staticmethod
     def fused_rows(nheads: int, kvheads: int, head_dim: int, vdim: int, values_are_keys: bool, gate) -> int:
@@ -165,6 +192,10 @@ class SinkAttention(Part):
             self._sink = self.tensor("sink").float().contiguous()
         elif self.sink_logit is not None:
             self._sink = torch.full((self.nheads,), self.sink_logit, dtype=torch.float32, device=device)
+        if self.has_distance:
+            self._distance = torch.stack([self.tensor("r1").float(), self.tensor("r2").float()], dim=1).contiguous()
+        if self.v_mix == "mixed":
+            self._mix = float(self.tensor("vmix").float().item())
         if self.norm_first:
             self._q_gain = self.tensor("q_norm").float().contiguous()
             self._k_gain = self.tensor("k_norm").float().contiguous()
@@ -172,15 +203,32 @@ class SinkAttention(Part):
     def cache_request(self):
         return KVRequest(self.kvheads, self.pad, self.window)
 
-    def heads_out(self, x, batch, cache_view, writes_cache: bool = True):
-        """The gated heads' results [tokens, nheads * vdim], before the output projection."""
-        proj = self.in_proj.forward(x)
+    def attend(self, proj, batch, cache_view, writes_cache: bool = True):
+        """The heads' results [tokens, nheads * pad] before gate and output projection, from the fused projection (the
+        first ``in_rows`` columns of ``proj``)."""
+        first = None
+        if self.v_mix == "first":
+            batch.scratch["first_values"] = (proj, self.value_col, self.kvheads * self.vdim)
+        elif self.v_mix == "mixed":
+            matrix, col, width = batch.scratch["first_values"]
+            if width != self.kvheads * self.vdim:
+                raise ValueError(f"sink_attention: {self.kvheads * self.vdim} values a token are mixed with {width}")
+            first = (matrix, col)
+        # queries that need nothing are read where the projection left them
+        in_place = (not self.rot_dims and not self.qk_norm and self.pad == self.head_dim
+                    and proj.shape[1] * proj.element_size() % 16 == 0)
         q = ops.qk_prepare_store(proj, self._inv_freq, self.rot_dims, self.qk_norm, self.eps, batch, cache_view,
                                  self.nheads, self.kvheads, self.head_dim, self.vdim, self.pad, writes_cache,
                                  norm_first=self.norm_first, q_gain=self._q_gain, k_gain=self._k_gain, halves=self.halves,
-                                 values_are_keys=self.values_are_keys, rot_mult=self.rot_mult)
-        o = ops.attention(q, batch, cache_view, self.nheads, self.kvheads, self.pad, self.scale, self.window, self._sink,
-                          chunk=self.chunk, softcap=self.softcap)
+                                 values_are_keys=self.values_are_keys, rot_mult=self.rot_mult, q_in_place=in_place,
+                                 first_values=first, v_mix=self._mix)
+        return ops.attention(proj if in_place else q, batch, cache_view, self.nheads, self.kvheads, self.pad, self.scale,
+                             self.window, self._sink, chunk=self.chunk, softcap=self.softcap, distance=self._distance)
+
+    def heads_out(self, x, batch, cache_view, writes_cache: bool = True):
+        """The gated heads' results [tokens, nheads * vdim], before the output projection."""
+        proj = self.in_proj.forward(x)
+        o = self.attend(proj, batch, cache_view, writes_cache)
         if not self.has_gate and self.pad == self.vdim and self.out_factor == 1.0:
             return o  # no gate, no padding to drop, no factor: the heads' results as attention left them
         return ops.sigmoid_gate(o, proj if self.has_gate else None, self.gate_col, self.nheads, self.vdim, self.pad,

@@ -23,6 +23,10 @@ feed-forward ends after its mixer.
 ``ParallelResidualBlock`` ("parallel_residual"): x += mixer(norm1(x)) + feed_forward(norm2(x)), both norms of the same
 stream and from one kernel; what it hands on is the list of its outputs with their factors.
 
+``JointParallelBlock`` ("parallel_joint"): x += mixer(h) + feed_forward(h) with ONE norm h = norm(x) that both read, made
+of two products: all that reads h is one matrix, all that is added to x another.  Then, where the layer has one, what it
+adds for the tokens themselves.
+
 ``OutputNormBlock`` ("output_norm"): a norm on each sublayer's output only, x += norm1(mixer(x));
 x += norm2(feed_forward(x)); the sublayers read the stream itself.  What it hands on is a ``NormedDelta`` as well; the
 kernel that adds it also leaves the summed stream in the compute dtype for the sublayer that reads it next.
@@ -32,8 +36,10 @@ from __future__ import annotations
 from ..config.specs import BlockSpec
 from .base import Part
 from ..kernels import ops
+from .linear import Linear
 from .norm import NormedDelta, StreamCopy
 from .registry import build_feed_forward, build_mixer, build_norm, register_block
+from .token_side import TokenSide
 
 
 class PreNormBlock(Part):
@@ -214,7 +220,60 @@ class ParallelResidualBlock(Part):
         return super().kernel_libraries(dtype) + ["elementwise"]
 
 
+class JointParallelBlock(Part):
+    """``parallel_joint``: h = norm(x); x += mixer(h) + feed_forward(h).  Both sublayers read the same h and both outputs go
+    into the same sum, so the layer has two products: [mixer's rows; feed-forward's rows] . h, and
+    [Wo | Wdown] . [heads' results | hidden values], whose sum over both is never rounded in between.  One kernel gates the
+    heads and activates the hidden values in between.  The mixer and the feed-forward are built with their projections
+    outside (``sink_attention`` with ``projections`` "outside"; ``projected_unit``, or ``routed_experts``, whose shared unit
+    takes the joint products while the routed ones stand beside them).  A layer may have no feed-forward.
+
+    ``token_side``: a ``TokenSide`` that follows; its output is then what stays pending."""
+
+    def __init__(self, spec: BlockSpec) -> None:
+        super().__init__()
+        n_norm, n_mixer, _, n_ff = spec.names
+        self.norm = self.add(n_norm, build_norm(spec.mixer_norm))
+        self.mixer = self.add(n_mixer, build_mixer(spec.mixer))
+        if getattr(self.mixer, "projects", True):
+            raise ValueError("a parallel_joint layer needs a mixer whose projections lie outside of it")
+        self.feed_forward = None
+        ff_rows = hidden = 0
+        if spec.feed_forward is not None:
+            ff = self.feed_forward = self.add(n_ff, build_feed_forward(spec.feed_forward))
+            if not hasattr(ff, "beside"):
+                raise ValueError("a parallel_joint layer needs a feed-forward that takes its rows from the joint projection")
+            ff_rows, hidden = ff.in_rows, ff.joint_hidden
+        self.hidden = hidden
+        dim = spec.mixer.dim
+        self.in_proj = self.add("in_proj", Linear(dim, self.mixer.in_rows + ff_rows))
+        self.out_proj = self.add("out_proj", Linear(self.mixer.out_columns + hidden, dim))
+        self.token_side = self.add("side", TokenSide(spec.token_side)) if spec.token_side is not None else None
+
+    def cache_request(self):
+        return self.mixer.cache_request()
+
+    def forward(self, residual, pending, batch, cache_view, writes_cache, dtype):
+        m, ff = self.mixer, self.feed_forward
+        h = self.norm.apply(residual, pending, dtype)
+        proj = self.in_proj.forward(h)
+        o = m.attend(proj, batch, cache_view, writes_cache)
+        z = ops.joint_activation(o, proj, m.gate_col if m.has_gate else -1, m.in_rows, m.nheads, m.vdim, m.pad, self.hidden,
+                                 ff.activation if ff is not None else 0, ff.gated if ff is not None else False)
+        parts = [(self.out_proj.forward(z), 1.0)]
+        beside = ff.beside(h) if ff is not None else None
+        if beside is not None:
+            parts.append((beside, 1.0))
+        if self.token_side is not None:
+            return self.token_side.forward(residual, parts, batch, dtype)
+        return ScaledParts(parts)
+
+    def kernel_libraries(self, dtype):
+        return super().kernel_libraries(dtype) + ["elementwise"]
+
+
 Block = PreNormBlock  # the name under which earlier callers know it
+register_block("parallel_joint", JointParallelBlock)
 register_block("parallel_residual", ParallelResidualBlock)
 register_block("output_norm", OutputNormBlock)
 register_block("post_norm", PostNormBlock)

@@ -7,6 +7,9 @@ Interface of an embedding (what the decoder calls):
 
 ``TableEmbedding`` ("table"): the token's row of the table (fms/models/llama.py:332).
 
+``PositionTableEmbedding`` ("table_and_positions"): the token's row plus a learned row of its position,
+e(t, p) = scale * table[t] + positions[p]; option ``positions``: how many there are.
+
 ``PairHashEmbedding`` ("pair_hash"): the token's row plus a row of a second, hashed table of token pairs,
 e(t) = table[token_t] + pairs[(token_(t-1) * mul_prev + token_t * mul_cur) mod buckets], and pairs[buckets] (the
 last row) for the first token of a sequence.  The token before a step's first row is the sequence's own state: one
@@ -39,6 +42,15 @@ class TableEmbedding(Part):
         return ["elementwise"]
 
 
+class PositionTableEmbedding(TableEmbedding):
+    def __init__(self, spec: EmbeddingSpec, vocab_size: int, dim: int) -> None:
+        super().__init__(spec, vocab_size, dim)
+        self.declare("positions", (int(dict(spec.options)["positions"]), dim), role="matrix")
+
+    def forward(self, batch, state_view, scale: float = 1.0):
+        return ops.embed_at(self.tensor("weight"), self.tensor("positions"), batch, scale)
+
+
 class PairHashEmbedding(TableEmbedding):
     def __init__(self, spec: EmbeddingSpec, vocab_size: int, dim: int) -> None:
         super().__init__(spec, vocab_size, dim)
@@ -59,4 +71,5 @@ class PairHashEmbedding(TableEmbedding):
 
 
 register_embedding("table", TableEmbedding)
+register_embedding("table_and_positions", PositionTableEmbedding)
 register_embedding("pair_hash", PairHashEmbedding)

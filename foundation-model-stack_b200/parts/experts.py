@@ -18,7 +18,14 @@ Further options, each of which leaves the above as it is when absent:
                               s + ``correction`` (a vector of the checkpoint, one number an expert, where ``correction``
                               is set); its weights are the chosen scores s (without the correction) over their sum
                               (+ 1e-20), times ``route_scale``; the weight multiplies the expert's OUTPUT
+    ``scoring`` "sigmoid_groups"  s = sigmoid(Wr h); the choice is by s + ``correction``, and the experts form ``groups``
+                              equal groups of neighbours of which the ``keep`` best can be chosen from (a group's score:
+                              the sum of its two largest choice scores); the weights are the chosen s as they are, times
+                              ``route_scale``, and multiply the experts' OUTPUTS
     ``unit`` "relu_squared"   expert_e(v) = Wdown,e relu(Wup,e v)^2: no gate; ``up`` [experts, hidden, dim]
+    ``unit`` "silu"           expert_e(v) = Wdown,e (silu(Wgate,e v) * Wup,e v)
+    ``shared`` spec           a further unit that runs for every token, a ``projected_unit`` whose products the block makes
+                              with its mixer's
 """
 from __future__ import annotations
 
@@ -26,7 +33,7 @@ from ..config.specs import FeedForwardSpec
 from ..kernels import ops
 from .base import Part
 from .linear import Linear
-from .registry import register_feed_forward
+from .registry import build_feed_forward, register_feed_forward
 
 
 class RoutedExperts(Part):
@@ -39,11 +46,21 @@ class RoutedExperts(Part):
         if not (0 < self.top <= self.experts) or self.hidden <= 0:
             raise ValueError(f"routed_experts: {self.experts} experts, top {self.top}, hidden {self.hidden}")
         self.scoring, self.unit = o.get("scoring", "sigmoid"), o.get("unit", "gated_clamped")
-        if self.scoring not in ("sigmoid", "softmax") or self.unit not in ("gated_clamped", "relu_squared"):
+        if (self.scoring not in ("sigmoid", "softmax", "sigmoid_groups")
+                or self.unit not in ("gated_clamped", "relu_squared", "silu")):
             raise ValueError(f"routed_experts: scoring {self.scoring!r}, unit {self.unit!r}")
         if self.unit == "gated_clamped" and "limit" not in o:
             raise ValueError("routed_experts: the gated unit needs its limit")
         self.route_scale, self.has_correction = float(o.get("route_scale", 1.0)), bool(o.get("correction", False))
+        self.groups, self.keep = int(o.get("groups", 1)), int(o.get("keep", 1))
+        if (self.groups <= 0 or self.experts % self.groups or not (0 < self.keep <= self.groups)
+                or self.keep * (self.experts // self.groups) < self.top):
+            raise ValueError(f"routed_experts: {self.experts} experts in {self.groups} groups of which {self.keep} stay, "
+                             f"top {self.top}")
+        shared = build_feed_forward(o["shared"]) if o.get("shared") is not None else None
+        self.in_rows = shared.in_rows if shared else 0
+        self.joint_hidden, self.activation = (shared.hidden, shared.activation) if shared else (0, 0)
+        self.gated = shared.gated if shared else False
         self.router = self.add("router", Linear(spec.dim, self.experts, False))
         if self.has_correction:
             self.declare("correction", (self.experts,), role="vector")
@@ -59,8 +76,20 @@ class RoutedExperts(Part):
         if self.has_correction:
             self._correction = self.tensor("correction").float().contiguous()
 
+    def beside(self, x):
+        """What a block that makes its sublayers' products together adds as it is: the routed experts."""
+        return self._routed(x)
+
     def forward(self, x):
-        if self.scoring == "softmax":
+        if self.in_rows:
+            raise ValueError("routed_experts: a shared unit belongs to a block that makes its products (parallel_joint)")
+        return self._routed(x)
+
+    def _routed(self, x):
+        if self.scoring == "sigmoid_groups":
+            routing = ops.route(x, self.router.tensor("weight"), self.top, ops.ROUTE_SIGMOID_GROUPS, self._correction,
+                                self.route_scale, self.groups, self.keep)
+        elif self.scoring == "softmax":
             routing = ops.route(x, self.router.tensor("weight"), self.top, ops.ROUTE_SOFTMAX, self._correction,
                                 self.route_scale)
         else:
@@ -68,11 +97,12 @@ class RoutedExperts(Part):
         if self.unit == "relu_squared":
             hidden = ops.routed_linear(routing.rows, self.tensor("up"), routing, relu_squared=True)
             return ops.route_gather(ops.routed_linear(hidden, self.tensor("down"), routing), routing)
-        hidden = ops.routed_linear(routing.rows, self.tensor("gate_up"), routing, True, self.limit, self.alpha)
+        hidden = ops.routed_linear(routing.rows, self.tensor("gate_up"), routing, True, self.limit, self.alpha,
+                                   silu=self.unit == "silu")
         return ops.route_gather(ops.routed_linear(hidden, self.tensor("down"), routing), routing)
 
     def kernel_libraries(self, dtype):
-        return ["grouped"]
+        return ["grouped", "elementwise"]
 
 
 register_feed_forward("routed_experts", RoutedExperts)

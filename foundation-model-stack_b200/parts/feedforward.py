@@ -5,7 +5,14 @@ Interface of a feed-forward (what a block calls):
 
     forward(x) -> y          x, y: [tokens, dim] in the compute dtype
 
-A feed-forward with routing would implement the same call and keep router and experts inside.
+A feed-forward with routing implements the same call and keeps router and experts inside.
+
+``ProjectedUnit`` ("projected_unit"): the hidden values of a feed-forward whose two products a block makes together with
+its mixer's (``JointParallelBlock``): act(up) of ``hidden`` columns, or, option ``gated``, act(gate) * up of twice as many.
+It has no tensors; what such a block asks of a feed-forward is
+
+    in_rows, joint_hidden, activation, gated       rows of the joint projection and what becomes of them
+    beside(x) -> y or None                         what it computes from the block's normed input by itself (routed experts)
 """
 from __future__ import annotations
 
@@ -16,6 +23,8 @@ from .linear import Linear
 from .registry import register_feed_forward
 
 ACTIVATIONS = {"silu": 0, "swish": 0, "gelu": 1, "gelu-tanh": 2, "gelu_pytorch_tanh": 2, "relu": 3}
+# for the kernels of ``ops.joint_activation`` and ``ops.token_gate``, which also know the square of relu
+UNGATED_ACTIVATIONS = dict(ACTIVATIONS, relu_squared=4)
 
 
 class GatedLinearUnit(Part):
@@ -37,4 +46,22 @@ class GatedLinearUnit(Part):
         return super().kernel_libraries(dtype) + ["elementwise"]
 
 
+class ProjectedUnit(Part):
+    def __init__(self, spec: FeedForwardSpec) -> None:
+        super().__init__()
+        act = spec.activation.lower()
+        if act not in UNGATED_ACTIVATIONS:
+            raise ValueError(f"activation {spec.activation!r} is not supported; supported: {sorted(UNGATED_ACTIVATIONS)}")
+        if spec.bias or spec.hidden <= 0:
+            raise ValueError(f"projected_unit: {spec.hidden} hidden values, bias {spec.bias}")
+        self.activation, self.hidden = UNGATED_ACTIVATIONS[act], int(spec.hidden)
+        self.joint_hidden = self.hidden
+        self.gated = bool(dict(spec.options).get("gated", False))
+        self.in_rows = self.hidden * (2 if self.gated else 1)
+
+    def beside(self, x):
+        return None
+
+
 register_feed_forward("glu", GatedLinearUnit)
+register_feed_forward("projected_unit", ProjectedUnit)

@@ -23,7 +23,8 @@ by value.
 the weight; adds several pending outputs with a factor each; ``apply_pair`` gives two norms of the same stream from
 one kernel.
 
-``LayerNorm`` ("layernorm"): y = (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * w, no bias.  Option
+``LayerNorm`` ("layernorm"): y = (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * w.  Option ``bias``: + b (a vector
+of the checkpoint; the norm of the stream only).  Option
 ``layer_scale``: a second vector ``scale`` multiplies the result element by element (the gain the kernel sees is
 w * scale, taken in float32 once).  It norms a sublayer's output on its way into the stream (as the ``norm`` of a
 ``NormedDelta``), and as a norm of the stream itself it adds what is pending and norms the sum in one kernel; with
@@ -71,12 +72,19 @@ class RMSNorm(Part):
         self.eps = float(spec.eps)
         self.offset = float(dict(spec.options).get("offset", 0.0))
         self.declare("weight", (spec.dim,), role="vector")
-        self._gain = None
+        self._gain = self._wide_gain = None
 
     def finalize(self, device, dtype) -> None:
         super().finalize(device, dtype)
         if self.offset != 0.0:
             self._gain = (self.tensor("weight").float() + self.offset).contiguous()
+        self._wide_gain = None
+
+    def mode_and_gain(self):
+        """(mode, float32 gain vector, eps): what ``ops.normed_add_norm`` takes."""
+        if self._wide_gain is None:
+            self._wide_gain = self.gain_vector().float().contiguous()
+        return ops.NORM_RMS, self._wide_gain, self.eps
 
     def gain_vector(self):
         return self._gain if self._gain is not None else self.tensor("weight")
@@ -135,10 +143,13 @@ class LayerNorm(Part):
         self.dim = spec.dim
         self.eps = float(spec.eps)
         self.layer_scale = bool(dict(spec.options).get("layer_scale", False))
+        self.has_bias = bool(dict(spec.options).get("bias", False))
         self.declare("weight", (spec.dim,), role="vector")
+        if self.has_bias:
+            self.declare("bias", (spec.dim,), role="vector")
         if self.layer_scale:
             self.declare("scale", (spec.dim,), role="vector")
-        self._gain = None
+        self._gain = self._bias = None
 
     def finalize(self, device, dtype) -> None:
         super().finalize(device, dtype)
@@ -146,14 +157,19 @@ class LayerNorm(Part):
         if self.layer_scale:
             g = g * self.tensor("scale").float()
         self._gain = g.contiguous()
+        if self.has_bias:
+            self._bias = self.tensor("bias").float().contiguous()
 
     def mode_and_gain(self):
-        """(mode, float32 gain vector, eps): what ``ops.normed_add_norm`` takes for either of its two norms."""
+        """(mode, float32 gain vector, eps): what ``ops.normed_add_norm`` takes for either of its two norms (its own bias
+        is handed over beside it where this is the norm of the stream)."""
         return ops.NORM_LAYER, self._gain, self.eps
 
     def add(self, residual, delta, out_dtype):
         """residual += this norm of ``delta`` (a sublayer's output), in float32; returns the stream in ``out_dtype``
         (the stream itself where that is float32)."""
+        if self.has_bias:
+            raise ValueError("a layer norm with a bias norms the stream, not an output on its way into it")
         if out_dtype == torch.float32:
             ops.normed_add_norm(residual, delta, self.mode_and_gain(), None, out_dtype, want_out=False)
             return residual
@@ -164,10 +180,12 @@ class LayerNorm(Part):
         if isinstance(delta, StreamCopy):
             delta = None
         if isinstance(delta, NormedDelta):
-            if not hasattr(delta.norm, "mode_and_gain"):
-                raise ValueError("a layer norm adds a pending output that is normed by a norm with mode_and_gain()")
+            if not hasattr(delta.norm, "mode_and_gain") or getattr(delta.norm, "has_bias", False):
+                raise ValueError("a layer norm adds a pending output that is normed by a norm with mode_and_gain() and no bias")
             delta, post = delta.delta, delta.norm.mode_and_gain()
-        return ops.normed_add_norm(residual, delta, post, self.mode_and_gain(), out_dtype, rows)
+        elif hasattr(delta, "parts"):  # several outputs with their factors
+            delta = list(delta.parts)
+        return ops.normed_add_norm(residual, delta, post, self.mode_and_gain(), out_dtype, rows, bias=self._bias)
 
     def kernel_libraries(self, dtype):
         return ["elementwise"]
