@@ -82,10 +82,14 @@ __device__ __forceinline__ int first_visible(const AttnArgs& a, int pos) {
 // by r' with r' * scale = softcap * tanh(r * scale / softcap).  tanh(x) = 1 - 2 / (exp(2 x) + 1) with the fast
 // exponential and division: its absolute error is a few 1e-7 (times the cap: far below what rounding the
 // probabilities to bfloat16 costs), it saturates to +-1 without a case of its own, and it costs a third of tanhf,
-// which doubled the tcgen05 prefill kernel's time (120 against 62 us for 2,048 tokens of 32 heads).
+// which doubled the tcgen05 prefill kernel's time (120 against 62 us for 2,048 tokens of 32 heads).  Exponential and
+// reciprocal are the one-instruction forms that flush denormals: those that do not cost a few instructions around each.
 __device__ __forceinline__ float capped_raw(const AttnArgs& a, float raw) {
-  const float t = __expf(2.f * raw * (a.scale / a.softcap));
-  return (1.f - __fdividef(2.f, t + 1.f)) * (a.softcap / a.scale);
+  float t, r;
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(t) : "f"(raw * (2.f * 1.4426950408889634f * (a.scale / a.softcap))));
+  asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(r) : "f"(t + 1.f));
+  const float c = a.softcap / a.scale;
+  return fmaf(-2.f * c, r, c);
 }
 
 // The distance term in the same units, r' with r' * scale = r1 * ln(1 + r2 * distance): `factor` is r1 * ln(2) / scale
@@ -95,8 +99,16 @@ __device__ __forceinline__ float2 distance_factor(const AttnArgs& a, int head) {
   const float2 r = a.distance[head];
   return make_float2(r.x * (0.69314718055994531f / a.scale), r.y);
 }
-__device__ __forceinline__ float distance_raw(float2 factor, int distance) {
-  return factor.x * __log2f(fmaf(factor.y, (float)distance, 1.f));
+// `origin` is distance_origin of some key's distance; `offset` (a compile-time number, so that no integer is converted)
+// says how many keys later the key at hand lies.
+__device__ __forceinline__ float distance_origin(float2 factor, int distance) { return fmaf(factor.y, (float)distance, 1.f); }
+__device__ __forceinline__ float log2_approx(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float less_distance(float raw, float2 factor, float origin, int offset) {
+  return fmaf(-factor.x, log2_approx(fmaf(-factor.y, (float)offset, origin)), raw);
 }
 
 // The cache block that holds key block kb of the sequence in `slot`; negative: none (a block given back behind a
@@ -636,7 +648,9 @@ static int attention_prefill(const void* q, void* out, int dtype, const void* ke
     if (make_map(&map_k, keys, rows, HD, BLK) || make_map(&map_v, values, rows, HD, BLK)) return 1;
     static bool configured_tc = false;
     if (!configured_tc) {
-      cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_SMEM);
+      cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_SMEM);
+      if (e == cudaSuccess)
+        e = cudaFuncSetAttribute(attn_prefill_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_SMEM);
       if (e != cudaSuccess) return fms_fail("attention_prefill: shared memory of %zu bytes refused: %s", TC_SMEM, cudaGetErrorString(e));
       configured_tc = true;
     }
@@ -644,8 +658,8 @@ static int attention_prefill(const void* q, void* out, int dtype, const void* ke
     const int gh = tc_heads_per_block(group);
     const long blocks = (long)n_tiles * kvheads * ((group + gh - 1) / gh);
     if (blocks > 0x7fffffffL) return fms_fail("attention_prefill: %ld thread blocks", blocks);
-    fms_launch(attn_prefill_tc_kernel, dim3((unsigned)blocks), dim3(192), TC_SMEM, stream, map_k, map_v, a, tiles, n_tiles,
-               error_flag);
+    fms_launch(a.distance ? attn_prefill_tc_kernel<true> : attn_prefill_tc_kernel<false>, dim3((unsigned)blocks), dim3(192), TC_SMEM,
+               stream, map_k, map_v, a, tiles, n_tiles, error_flag);
     return fms_launch_status("attention_prefill");
   }
 #endif

@@ -261,10 +261,11 @@ __global__ void __launch_bounds__(NW * 32, WK == 32 ? 16 / NW : 12 / NW)
         for (int e = 0; e < 4; ++e) st[t][e] = capped_raw(a, st[t][e]);
     }
     if (a.distance) {
+      const float origin[2] = {distance_origin(dist[0], pos - first - g), distance_origin(dist[1], pos - first - g)};
 #pragma unroll
       for (int t = 0; t < WT; ++t)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) st[t][e] -= distance_raw(dist[e & 1], pos - (first + 16 * t + g + 8 * (e >> 1)));
+        for (int e = 0; e < 4; ++e) st[t][e] = less_distance(st[t][e], dist[e & 1], origin[e & 1], 16 * t + 8 * (e >> 1));
     }
     if (!whole) {
 #pragma unroll
@@ -506,11 +507,12 @@ __global__ void __launch_bounds__(PF_WARPS * 32, HD <= 128 ? 3 : 1) attn_prefill
         for (int e = 0; e < 4; ++e) s[j][e] = capped_raw(a, s[j][e]);
     }
     if (a.distance) {
+      const float origin[2] = {distance_origin(dist[0], row_pos[0] - kb * BLK - 2 * c),
+                               distance_origin(dist[1], row_pos[1] - kb * BLK - 2 * c)};
 #pragma unroll
       for (int j = 0; j < 8; ++j)
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-          s[j][e] -= distance_raw(dist[e >> 1], row_pos[e >> 1] - (kb * BLK + 8 * j + 2 * c + (e & 1)));
+        for (int e = 0; e < 4; ++e) s[j][e] = less_distance(s[j][e], dist[e >> 1], origin[e >> 1], 8 * j + (e & 1));
     }
     float tile_max[2] = {-INFINITY, -INFINITY};
 #pragma unroll

@@ -201,10 +201,11 @@ __global__ void __launch_bounds__((SR_WARPS + 1) * 32, 1)
           dist[h] = 2 * c + h < ng ? distance_factor(a, kvh * group + g0 + 2 * c + h) : make_float2(0.f, 0.f);
         pos = a.len_after[seq] - 1;
       }
+      const float origin[2] = {distance_origin(dist[0], pos - kb * BLK - g), distance_origin(dist[1], pos - kb * BLK - g)};
 #pragma unroll
       for (int t = 0; t < 4; ++t)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) st[t][e] -= distance_raw(dist[e & 1], pos - (kb * BLK + 16 * t + g + 8 * (e >> 1)));
+        for (int e = 0; e < 4; ++e) st[t][e] = less_distance(st[t][e], dist[e & 1], origin[e & 1], 16 * t + 8 * (e >> 1));
     }
     if (!whole) {
 #pragma unroll

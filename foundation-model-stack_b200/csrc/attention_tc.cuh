@@ -29,6 +29,17 @@ constexpr int TC_Q_BYTES = TC_ROWS * HD * 2;
 constexpr size_t TC_SMEM = 1024 + TC_Q_BYTES + (size_t)TC_STAGES * 2 * TC_KV_TILE + 256;  // two blocks fit an SM
 constexpr int TC_TMEM_COLS = HD + 2 * BLK <= 128 ? 128 : 256;  // O: HD columns, S: two buffers of 64 columns
 
+// The distance term of a block of keys is the same for rows and keys equally far apart, so a warp (32 rows: positions x
+// heads of a block, TC_DIST_HEADS at most) makes a table of it, one value a head and distance, instead of one logarithm a
+// score.  Row (position p, head h) and key j read entry h * stride + p - (the warp's first position) + 63 - j; the stride
+// sends the heads of a position to different banks.
+constexpr int TC_DIST_HEADS = 8;
+constexpr int TC_DIST_FLOATS = 800;  // at most heads * stride
+__device__ __forceinline__ int tc_distance_stride(int gh) {
+  const int span = BLK - 1 + 31 / gh + 2, want = 32 / gh % 32;
+  return span + ((want - span) % 32 + 32) % 32;
+}
+
 // 2^x in one special-function instruction (relative error about 2^-22; 0 for -inf)
 __device__ __forceinline__ float fast_exp2(float x) {
   float y;
@@ -39,6 +50,8 @@ __device__ __forceinline__ float fast_exp2(float x) {
 __host__ __device__ inline int tc_heads_per_block(int group) { return group < TC_ROWS ? group : TC_ROWS; }
 __host__ __device__ inline int tc_positions_per_block(int group) { return TC_ROWS / tc_heads_per_block(group); }
 
+// DISTANCE: the kernel for calls with a distance term (the others have neither its table nor its registers)
+template <bool DISTANCE>
 __global__ void __launch_bounds__(192, 2) attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k,
                                                                  const __grid_constant__ CUtensorMap map_v, AttnArgs a,
                                                                  const int* __restrict__ tiles, int n_tiles,
@@ -59,6 +72,8 @@ __global__ void __launch_bounds__(192, 2) attn_prefill_tc_kernel(const __grid_co
   uint64_t* q_ready = o_done + 2;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(q_ready + 1);
   __shared__ int failed_flag;
+  __shared__ float distance_table[DISTANCE ? 4 : 1][DISTANCE ? TC_DIST_FLOATS : 1];
+  __shared__ float2 distance_factors[DISTANCE ? TC_DIST_HEADS : 1];
   volatile int* failed = &failed_flag;
   pdl_launch_dependents();
 
@@ -187,11 +202,31 @@ __global__ void __launch_bounds__(192, 2) attn_prefill_tc_kernel(const __grid_co
       mbar_arrive(q_ready);
     }
     const float scale2 = a.scale * LOG2E;
-    const float2 dist = a.distance && row_ok ? distance_factor(a, kvh * group + g0 + gi) : make_float2(0.f, 0.f);
+    const bool tabled = DISTANCE && gh <= TC_DIST_HEADS;
+    if (tabled && r < ng) distance_factors[r] = distance_factor(a, kvh * group + g0 + r);
+    if (DISTANCE) asm volatile("bar.sync 1, 128;\n" ::: "memory");  // the four warps of this branch, once
+    const int stride = tc_distance_stride(gh), pi_first = quarter * 32 / gh, span = (quarter * 32 + 31) / gh - pi_first + BLK;
+    float* table = distance_table[DISTANCE ? quarter : 0];
+    const float* my_table = table + gi * stride + pi - pi_first;  // key j at [BLK - 1 - j]
     float m_ref = -INFINITY, l = 0.f;  // the exponents are taken against m_ref (base 2); l is the sum of them
     bool ok = true;
     for (int i = 0; i < nblocks && ok; ++i) {
       const int kb = kb_lo + i, s = i % TC_STAGES;
+      const int blk = block_of(a, slot, kb);  // asked for here: it is needed after the exponentials
+      if (tabled) {  // while the scores are on their way; distances of keys after a row count as 0 (they are masked)
+        __syncwarp();
+        float away[3];  // the distances of this lane's entries, at most 96 a head
+#pragma unroll
+        for (int k = 0; k < 3; ++k) away[k] = (float)max(p_first + pi_first - kb * BLK - (BLK - 1) + lane + 32 * k, 0);
+#pragma unroll 4
+        for (int h = 0; h < ng; ++h) {
+          const float2 f = distance_factors[h];
+#pragma unroll
+          for (int k = 0; k < 3; ++k)
+            if (lane + 32 * k < span) table[h * stride + lane + 32 * k] = f.x * log2_approx(fmaf(f.y, away[k], 1.f));
+        }
+        __syncwarp();
+      }
       ok = __all_sync(0xffffffffu, wait_or_abort(&s_full[i & 1], (i >> 1) & 1, failed));  // the same decision in
       if (!ok) break;                                                    // every lane: tensor-memory loads are warp-wide
       tc_fence_after();
@@ -201,13 +236,21 @@ __global__ void __launch_bounds__(192, 2) attn_prefill_tc_kernel(const __grid_co
       // raw scores; the scale (positive) goes into the exponent's multiply-add.  A block that every row of the tile
       // sees whole needs no mask; rows without a query hold zeros there and are never stored.
       const bool whole = kb * BLK + BLK - 1 <= p_first && kb * BLK >= first_visible(a, p_last);
-      if (a.softcap > 0.f) {
+      if (tabled && a.softcap > 0.f) {  // both in one pass: the table's loads beside the exponentials
+#pragma unroll
+        for (int j = 0; j < BLK; ++j) sc[j] = capped_raw(a, sc[j]) - my_table[BLK - 1 - j];
+      } else if (a.softcap > 0.f) {
 #pragma unroll
         for (int j = 0; j < BLK; ++j) sc[j] = capped_raw(a, sc[j]);
-      }
-      if (a.distance) {
+      } else if (tabled) {
 #pragma unroll
-        for (int j = 0; j < BLK; ++j) sc[j] -= distance_raw(dist, my_pos - (kb * BLK + j));
+        for (int j = 0; j < BLK; ++j) sc[j] -= my_table[BLK - 1 - j];
+      }
+      if (DISTANCE && !tabled) {
+        const float2 dist = row_ok ? distance_factor(a, kvh * group + g0 + gi) : make_float2(0.f, 0.f);
+        const float origin = distance_origin(dist, my_pos - kb * BLK);
+#pragma unroll
+        for (int j = 0; j < BLK; ++j) sc[j] = less_distance(sc[j], dist, origin, j);
       }
       if (!whole) {
 #pragma unroll
@@ -258,7 +301,6 @@ __global__ void __launch_bounds__(192, 2) attn_prefill_tc_kernel(const __grid_co
       const float psum = (ps[0] + ps[1]) + (ps[2] + ps[3]);
       l += psum;
       // the values of a block that the sequence fills only partly: rows beyond its length become zeros
-      const int blk = block_of(a, slot, kb);
       if (kb * BLK + BLK > len || blk < 0) {
         ok = __all_sync(0xffffffffu, wait_or_abort(&v_full[s], (i / TC_STAGES) & 1, failed));
         if (!ok) break;

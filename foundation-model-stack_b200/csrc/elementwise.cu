@@ -594,7 +594,8 @@ FMS_API int fms_normed_add_norm(float* residual, const void* d0, float s0, const
   bool four = dim % 4 == 0 && (uintptr_t)residual % 16 == 0 && (uintptr_t)out % (4 * item) == 0 && (uintptr_t)gain % 16 == 0 &&
               (uintptr_t)post_gain % 16 == 0 && (uintptr_t)bias % 16 == 0;
   for (int k = 0; k < 4; ++k) four = four && (uintptr_t)parts.d[k] % (4 * item) == 0;
-  const int threads = dim >= 8192 ? 1024 : (dim >= 2048 ? 512 : (dim >= 1024 ? 256 : 128));
+  int threads = dim >= 8192 ? 1024 : (dim >= 2048 ? 512 : (dim >= 1024 ? 256 : 128));
+  if (n_rows <= 148 && threads < 1024 && dim > 4 * threads) threads *= 2;  // few rows: the shortest chain a row can have
   const int nper = (dim + threads - 1) / threads;
 #define FMS_NAN(NPER, VEC)                                                                                                  \
   FMS_DISPATCH_DTYPE(dtype, T, fms_launch(normed_add_norm_kernel<T, NPER, VEC>, dim3(n_rows), dim3(threads), 0, stream,     \
@@ -710,8 +711,17 @@ FMS_API int fms_token_gate(const void* z, int dtype, const void* table, const in
 //   out[t, h * vdim + e]      = o[t, h * pad + e] * sigmoid(proj[t, gate_col + h * vdim + e])      (gate_col < 0: no gate)
 //   out[t, nheads * vdim + f] = act(proj[t, ff_col + f])                                           ff_gated 0
 //                             = act(proj[t, ff_col + f]) * proj[t, ff_col + hidden + f]            ff_gated 1
-// VEC values a thread (4 where sizes and addresses allow accesses of 4 values, else 1)
+// VEC values a thread (8 or 4 where sizes and addresses allow such accesses, else 1)
 // ---------------------------------------------------------------------------------------------------
+// bfloat16 results take the fast exponential and division (relative errors near 2^-22 before rounding)
+template <typename T> __device__ __forceinline__ float sigmoid_for(float g) { return 1.f / (1.f + expf(-g)); }
+template <> __device__ __forceinline__ float sigmoid_for<__nv_bfloat16>(float g) { return __fdividef(1.f, 1.f + __expf(-g)); }
+template <typename T, int VEC> __device__ __forceinline__ void load_values(const T* p, float (&x)[VEC]) {
+  if constexpr (VEC == 8) embed_load8(p, x);
+  else if constexpr (VEC == 4) ldv4(p, x);
+  else x[0] = to_f32(*p);
+}
+
 template <typename T, int VEC>
 __global__ void joint_activation_kernel(const T* o, const T* proj, int stride, int gate_col, int ff_col, T* out, int nheads,
                                         int vdim, int pad, int hidden, int act, int ff_gated, size_t total) {
@@ -724,30 +734,37 @@ __global__ void joint_activation_kernel(const T* o, const T* proj, int stride, i
   const int c = (int)(i - t * width);
   const T* row = proj + t * stride;
   float v[VEC], g[VEC];
-  auto load = [](const T* p, float (&x)[VEC]) {
-    if constexpr (VEC == 4) ldv4(p, x);
-    else x[0] = to_f32(*p);
-  };
   if (c < heads_w) {
     const int h = c / vdim, e = c - h * vdim;
-    load(o + (t * nheads + h) * pad + e, v);
+    load_values<T, VEC>(o + (t * nheads + h) * pad + e, v);
     if (gate_col >= 0) {
-      load(row + gate_col + c, g);
+      load_values<T, VEC>(row + gate_col + c, g);
 #pragma unroll
-      for (int k = 0; k < VEC; ++k) v[k] *= 1.f / (1.f + expf(-g[k]));
+      for (int k = 0; k < VEC; ++k) v[k] *= sigmoid_for<T>(g[k]);
     }
   } else {
-    load(row + ff_col + (c - heads_w), v);
+    load_values<T, VEC>(row + ff_col + (c - heads_w), v);
 #pragma unroll
-    for (int k = 0; k < VEC; ++k) v[k] = activate(v[k], act);
+    for (int k = 0; k < VEC; ++k) v[k] = act == 0 ? v[k] * sigmoid_for<T>(v[k]) : activate(v[k], act);
     if (ff_gated) {
-      load(row + ff_col + hidden + (c - heads_w), g);
+      load_values<T, VEC>(row + ff_col + hidden + (c - heads_w), g);
 #pragma unroll
       for (int k = 0; k < VEC; ++k) v[k] *= g[k];
     }
   }
-  if constexpr (VEC == 4) stv4(out + i, v);
-  else out[i] = from_f32<T>(v[0]);
+  if constexpr (VEC == 1) {
+    out[i] = from_f32<T>(v[0]);
+  } else if constexpr (VEC == 4) {
+    stv4(out + i, v);
+  } else if constexpr (sizeof(T) == 2) {
+    uint32_t w[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const __nv_bfloat162 b = __floats2bfloat162_rn(v[2 * k], v[2 * k + 1]);
+      w[k] = *reinterpret_cast<const uint32_t*>(&b);
+    }
+    *reinterpret_cast<uint4*>(out + i) = make_uint4(w[0], w[1], w[2], w[3]);
+  }
 }
 
 FMS_API int fms_joint_activation(const void* o, const void* proj, int stride, int gate_col, int ff_col, void* out, int dtype,
@@ -758,14 +775,20 @@ FMS_API int fms_joint_activation(const void* o, const void* proj, int stride, in
     return fms_fail("joint_activation: %d heads of %d (%d), %d hidden values, activation %d", nheads, vdim, pad, hidden, act);
   const size_t total = (size_t)n_tokens * (nheads * vdim + hidden);
   const size_t item = dtype == FMS_BF16 ? 2 : 4;
-  const bool four = vdim % 4 == 0 && pad % 4 == 0 && hidden % 4 == 0 && stride % 4 == 0 && (gate_col < 0 || gate_col % 4 == 0) &&
-                    (hidden == 0 || ff_col % 4 == 0) && (uintptr_t)o % (4 * item) == 0 && (uintptr_t)out % (4 * item) == 0 &&
-                    (uintptr_t)proj % (4 * item) == 0;
+  auto runs_of = [&](int n) {
+    return vdim % n == 0 && pad % n == 0 && hidden % n == 0 && stride % n == 0 && (gate_col < 0 || gate_col % n == 0) &&
+           (hidden == 0 || ff_col % n == 0) && (uintptr_t)o % (n * item) == 0 && (uintptr_t)out % (n * item) == 0 &&
+           (uintptr_t)proj % (n * item) == 0;
+  };
 #define FMS_JOINT(VEC)                                                                                                       \
   FMS_DISPATCH_DTYPE(dtype, T, fms_launch(joint_activation_kernel<T, VEC>, dim3((unsigned)((total / VEC + 255) / 256)), dim3(256), \
                                           0, stream, (const T*)o, (const T*)proj, stride, gate_col, ff_col, (T*)out, nheads, vdim, \
                                           pad, hidden, act, ff_gated, total))
-  if (four) FMS_JOINT(4);
+  if (dtype == FMS_BF16 && runs_of(8))
+    fms_launch(joint_activation_kernel<__nv_bfloat16, 8>, dim3((unsigned)((total / 8 + 255) / 256)), dim3(256), 0, stream,
+               (const __nv_bfloat16*)o, (const __nv_bfloat16*)proj, stride, gate_col, ff_col, (__nv_bfloat16*)out, nheads, vdim, pad,
+               hidden, act, ff_gated, total);
+  else if (runs_of(4)) FMS_JOINT(4);
   else FMS_JOINT(1);
 #undef FMS_JOINT
   return fms_launch_status("joint_activation");

@@ -18,6 +18,9 @@
 //   GLU8:   rows r..r+7 of the gate and of the up matrix of a fused [gate; up] weight; the epilogue writes
 //           act(gate) * up (fms/modules/feedforward.py:291-292) without the [M, 2 hidden] round trip.
 //
+// GROUPED: the rows of x are sorted into groups (offsets on the device), each with a matrix of its own, and a block belongs
+// to one group (blockIdx.y); a group's rows are at most 8 and a group without rows reads nothing.
+//
 // The weights of the first ring stages are requested before the kernel waits for the kernel before it
 // (programmatic dependent launch): weights do not depend on it, so the stream of weights from memory does
 // not stop between the kernels of a step.
@@ -42,6 +45,15 @@ struct RopeArgs {
   int table_stride, block_tokens, nheads, kvheads, head_dim, write_cache;
   int* error_flag;
   int n_seqs, table_rows, pool_blocks;  // extents of slots, of the table and of the cache, for the bounds-checked build
+};
+
+// What the ROWS16 epilogue does beyond the product: nothing, or y = act(v) * table[tokens[m]] (table set), or the square of
+// relu (squares).  offsets: GROUPED only.
+struct RowArgs {
+  const __nv_bfloat16* table;  // [vocab, N]
+  const int* tokens;           // [M]
+  int vocab, squares;
+  const int* offsets;          // [groups + 1]
 };
 
 __device__ __forceinline__ void mma_bf16(float* d, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
@@ -75,12 +87,12 @@ __device__ __forceinline__ float activate(float g, int act) {
 }
 
 // NT: tiles of 8 batch rows (M <= 8 NT).  RT: tiles per block.  D: ring stages.
-template <int NT, int RT, int MODE, int D, typename TOut>
+template <int NT, int RT, int MODE, int D, typename TOut, bool GROUPED>
 __global__ void __launch_bounds__(THREADS) linear_skinny_kernel(const __nv_bfloat16* __restrict__ x,
                                                                 const __nv_bfloat16* __restrict__ w,
                                                                 const __nv_bfloat16* __restrict__ bias,
                                                                 TOut* __restrict__ y, int M, int N, int K, int hidden,
-                                                                int act, RopeArgs rope) {
+                                                                int act, RopeArgs rope, RowArgs extra) {
   constexpr int HALVES = 2;                           // weight rows a lane reads per tile
   constexpr int TILE_ROWS = MODE == GLU8 ? 8 : 16;    // output rows (or gate/up pairs) per tile
   constexpr int WL = RT * HALVES;                     // weight pieces per stage
@@ -91,6 +103,15 @@ __global__ void __launch_bounds__(THREADS) linear_skinny_kernel(const __nv_bfloa
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int g = lane >> 2, c = lane & 3;
   const int n_rows = MODE == GLU8 ? 2 * hidden : N;  // rows of w
+  if (GROUPED) {  // which weights are read depends on the kernel before
+    pdl_wait();
+    const int r_lo = __ldcg(extra.offsets + blockIdx.y), r_hi = __ldcg(extra.offsets + blockIdx.y + 1);
+    M = min(r_hi - r_lo, 8 * NT);
+    if (M <= 0) return;  // the whole block
+    x += (size_t)r_lo * K;
+    w += (size_t)blockIdx.y * n_rows * K;
+    y += (size_t)r_lo * (MODE == GLU8 ? hidden : N);
+  }
 
   const __nv_bfloat16* wp[RT][2];
 #pragma unroll
@@ -142,7 +163,7 @@ __global__ void __launch_bounds__(THREADS) linear_skinny_kernel(const __nv_bfloa
 #pragma unroll
   for (int i = 0; i < D; ++i) issue_w(i);  // weights: before the wait for the kernel that produces x
   cp_async_commit();
-  pdl_wait();
+  if (!GROUPED) pdl_wait();
 #pragma unroll
   for (int i = 0; i < D; ++i) issue_x(i);
   cp_async_commit();
@@ -258,19 +279,26 @@ __global__ void __launch_bounds__(THREADS) linear_skinny_kernel(const __nv_bfloa
       if (row < N && m < M) {
         float v = red[0][t][j][l][e];
         if (bias) v += __bfloat162float(bias[row]);
+        if (extra.table) {
+          const int tok = __ldcg(extra.tokens + m);  // a token outside the vocabulary: the embedding has set the flag
+          v = tok >= 0 && tok < extra.vocab ? activate(v, act) * __bfloat162float(extra.table[(size_t)tok * N + row]) : 0.f;
+        } else if (extra.squares) {
+          v = fmaxf(v, 0.f);
+          v *= v;
+        }
         if (FMS_IN((size_t)m * N + row, (size_t)M * N)) y[(size_t)m * N + row] = from_f32<TOut>(v);
       }
     }
   }
 }
 
-template <int NT, int RT, int MODE, typename TOut>
+template <int NT, int RT, int MODE, typename TOut, bool GROUPED = false>
 int launch_typed(const void* x, const void* w, const void* bias, void* y, int M, int N, int K, int hidden, int act,
-                 cudaStream_t stream, const RopeArgs& rope = RopeArgs{}) {
+                 cudaStream_t stream, const RopeArgs& rope = RopeArgs{}, const RowArgs& extra = RowArgs{}, int groups = 1) {
   constexpr int LOADS = RT * 2 + NT;
   constexpr int D = LOADS <= 2 ? 7 : (LOADS == 3 ? 5 : (LOADS == 4 ? 4 : 3));  // 56 to 72 KB of ring per block
   constexpr size_t smem = (size_t)D * LOADS * THREADS * sizeof(uint4);
-  auto kernel = linear_skinny_kernel<NT, RT, MODE, D, TOut>;
+  auto kernel = linear_skinny_kernel<NT, RT, MODE, D, TOut, GROUPED>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -280,8 +308,8 @@ int launch_typed(const void* x, const void* w, const void* bias, void* y, int M,
   constexpr int TILE_ROWS = MODE == GLU8 ? 8 : 16;
   const int rows = MODE == GLU8 ? hidden : N;
   const int blocks = (rows + TILE_ROWS * RT - 1) / (TILE_ROWS * RT);
-  cudaError_t e = fms_launch(kernel, dim3(blocks), dim3(THREADS), smem, stream, (const __nv_bfloat16*)x,
-                             (const __nv_bfloat16*)w, (const __nv_bfloat16*)bias, (TOut*)y, M, N, K, hidden, act, rope);
+  cudaError_t e = fms_launch(kernel, dim3(blocks, groups), dim3(THREADS), smem, stream, (const __nv_bfloat16*)x,
+                             (const __nv_bfloat16*)w, (const __nv_bfloat16*)bias, (TOut*)y, M, N, K, hidden, act, rope, extra);
   if (e != cudaSuccess) return fms_fail("linear_bf16_skinny: launch failed: %s", cudaGetErrorString(e));
   return 0;
 }
@@ -308,6 +336,30 @@ FMS_API int fms_linear_bf16_skinny(const void* x, const void* w, const void* bia
   // very many weight rows: 32 rows a block, which halves the re-reading of x
   if (N < 16384) return launch<1, 1, ROWS16>(x, w, bias, y, out_dtype, M, N, K, 0, 0, stream);
   return launch<1, 2, ROWS16>(x, w, bias, y, out_dtype, M, N, K, 0, 0, stream);
+}
+
+// y [M, N] = act(x w[N, K]^T) * table[tokens[m], :]: a small product gated by the tokens' own rows of a table [vocab, N].
+FMS_API int fms_token_gate_bf16_skinny(const void* x, const void* w, const void* table, const int* tokens, void* y, int M, int N,
+                                       int K, int vocab, int act, cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (M > 8) return fms_fail("token_gate_bf16_skinny: %d rows, at most 8", M);
+  if (K <= 0 || K % 8 || vocab <= 0 || act < 0 || act > 3 || !table || !tokens)
+    return fms_fail("token_gate_bf16_skinny: K %d, vocabulary %d, activation %d", K, vocab, act);
+  const RowArgs extra{(const __nv_bfloat16*)table, tokens, vocab, 0, nullptr};
+  return launch_typed<1, 1, ROWS16, __nv_bfloat16>(x, w, nullptr, y, M, N, K, 0, act, stream, RopeArgs{}, extra);
+}
+
+// Groups of at most 8 rows: for the rows offsets[g] .. offsets[g + 1] of x [rows, K], w [groups, N (or 2 N), K],
+// kind 0: y = x w^T; 2: its square where positive, else 0; 3: silu(gate) * up with w[g] = [gate; up].  y [rows, N].
+FMS_API int fms_grouped_bf16_skinny(const void* x, const void* w, void* y, const int* offsets, int groups, int N, int K, int kind,
+                                    cudaStream_t stream) {
+  if (groups <= 0 || N <= 0) return 0;
+  if (groups > 65535 || K <= 0 || K % 8 || !offsets || (kind != 0 && kind != 2 && kind != 3))
+    return fms_fail("grouped_bf16_skinny: %d groups, K %d, kind %d", groups, K, kind);
+  const RowArgs extra{nullptr, nullptr, 0, kind == 2 ? 1 : 0, offsets};
+  if (kind == 3)
+    return launch_typed<1, 2, GLU8, __nv_bfloat16, true>(x, w, nullptr, y, 8, 2 * N, K, N, 0, stream, RopeArgs{}, extra, groups);
+  return launch_typed<1, 1, ROWS16, __nv_bfloat16, true>(x, w, nullptr, y, 8, N, K, 0, 0, stream, RopeArgs{}, extra, groups);
 }
 
 // The fused projection of an attention layer for up to 8 tokens: [q | k | v] = x [M, K] w[(nheads + 2 kvheads) head_dim, K]^T

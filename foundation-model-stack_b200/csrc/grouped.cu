@@ -151,6 +151,20 @@ __device__ __forceinline__ void rows_load8(const __nv_bfloat16* p, float* v) {
   }
 }
 
+__device__ __forceinline__ void rows_store8(float* p, const float* v) {
+  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+__device__ __forceinline__ void rows_store8(__nv_bfloat16* p, const float* v) {
+  uint32_t o[4];
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const __nv_bfloat162 b = __floats2bfloat162_rn(v[2 * k], v[2 * k + 1]);
+    o[k] = *reinterpret_cast<const uint32_t*>(&b);
+  }
+  *reinterpret_cast<uint4*>(p) = make_uint4(o[0], o[1], o[2], o[3]);
+}
+
 // pieces of a weight row that a lane of the row-walking kernel has in flight for an ungated product.  Measured through
 // decode steps of 8 sequences over four layers with 16 experts of 3,584: one piece 2.00 ms, two 1.67, four 2.85 (the
 // registers of four pieces and of their rows of x cost more blocks a multiprocessor than the loads in flight gain)
@@ -289,40 +303,15 @@ __global__ void gated_clamped_vec_kernel(const __nv_bfloat16* gu, __nv_bfloat16*
 }
 
 // ---- routing -----------------------------------------------------------------------------------------
-// One block per token.  logits in shared memory; warp 0 then takes the `top` largest one after the other.
-constexpr int ROUTE_WARPS = 8;
+// One block per token: logits in shared memory, a warp per expert at a time (vec != 0: rows of a multiple of 8 values on 16
+// bytes, 8 values a lane and load); warp 0 then chooses.  With `logits` (another product has made them: many tokens) only
+// the choice is left, a warp per token.
+constexpr int ROUTE_WARPS = 16, CHOOSE_WARPS = 8;
 
-template <typename T, typename TW>
-__global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(const T* __restrict__ x, const TW* __restrict__ router,
-                                                    int* __restrict__ expert, float* __restrict__ weight,
-                                                    int dim, int experts, int top, int mode,
-                                                    const float* __restrict__ correction, float route_scale, int groups,
-                                                    int keep) {
-  extern __shared__ float sm[];  // dim values of x, `experts` logits, `experts` scores (mode 1, 2), `groups` scores (mode 2)
-  float* xs = sm;
-  float* logit = sm + dim;
-  float* score = logit + experts;
-  pdl_launch_dependents();
-  pdl_wait();
-  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int d = threadIdx.x; d < dim; d += blockDim.x) xs[d] = to_f32(x[(size_t)t * dim + d]);
-  __syncthreads();
-  for (int e = warp; e < experts; e += ROUTE_WARPS) {
-    const TW* wr = router + (size_t)e * dim;
-    float a = 0.f, b = 0.f, c = 0.f, d4 = 0.f;  // four chains: the loads of one do not wait for another's sum
-    int d = lane;
-    for (; d + 96 < dim; d += 128) {
-      a = fmaf(xs[d], to_f32(wr[d]), a);
-      b = fmaf(xs[d + 32], to_f32(wr[d + 32]), b);
-      c = fmaf(xs[d + 64], to_f32(wr[d + 64]), c);
-      d4 = fmaf(xs[d + 96], to_f32(wr[d + 96]), d4);
-    }
-    for (; d < dim; d += 32) a = fmaf(xs[d], to_f32(wr[d]), a);
-    a = warp_sum((a + b) + (c + d4));
-    if (lane == 0) logit[e] = a;
-  }
-  __syncthreads();
-  if (warp != 0) return;
+// What a warp does with one token's logits (in shared memory, `score` behind them: experts + groups values of scratch).
+__device__ __forceinline__ void route_choose(float* logit, float* score, int* expert, float* weight, int experts, int top, int mode,
+                             const float* correction, float route_scale, int groups, int keep) {
+  const int lane = threadIdx.x & 31;
   if (mode == 1) {
     // scores = softmax over all experts; the choice is by score + correction, the weights are the chosen scores over
     // their sum (+ 1e-20), times route_scale
@@ -398,8 +387,8 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(const T* __rest
     }
     if (at >= experts) at = k;  // every logit was NaN or -inf: any expert, so that nothing below reads outside
     if (lane == 0) {
-      expert[(size_t)t * top + k] = at;
-      weight[(size_t)t * top + k] = mode == 1 ? score[at] : (mode == 2 ? score[at] * route_scale : 1.f / (1.f + expf(-best)));
+      expert[k] = at;
+      weight[k] = mode == 1 ? score[at] : (mode == 2 ? score[at] * route_scale : 1.f / (1.f + expf(-best)));
       logit[at] = -INFINITY;
     }
     if (mode == 1) picked_sum += score[at];
@@ -407,8 +396,80 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(const T* __rest
   }
   if (mode == 1 && lane == 0) {
     const float f = route_scale / (picked_sum + 1e-20f);
-    for (int k = 0; k < top; ++k) weight[(size_t)t * top + k] *= f;
+    for (int k = 0; k < top; ++k) weight[k] *= f;
   }
+}
+
+template <typename T, typename TW>
+__global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(const T* x, const TW* router, int* expert, float* weight, int dim,
+                                                                 int experts, int top, int mode, const float* correction,
+                                                                 float route_scale, int groups, int keep, int vec) {
+  extern __shared__ float sm[];  // dim values of x, `experts` logits, `experts` scores (mode 1, 2), `groups` scores (mode 2)
+  float* xs = sm;
+  float* logit = sm + dim;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (vec) {
+    for (int d = 8 * threadIdx.x; d < dim; d += 8 * blockDim.x) {
+      float v[8];
+      rows_load8(x + (size_t)t * dim + d, v);
+      rows_store8(xs + d, v);
+    }
+  } else {
+    for (int d = threadIdx.x; d < dim; d += blockDim.x) xs[d] = to_f32(x[(size_t)t * dim + d]);
+  }
+  __syncthreads();
+  for (int e = warp; e < experts; e += ROUTE_WARPS) {
+    const TW* wr = router + (size_t)e * dim;
+    float a = 0.f, b = 0.f, c = 0.f, d4 = 0.f;  // four chains: the loads of one do not wait for another's sum
+    if (vec) {
+      for (int d0 = 8 * lane; d0 < dim; d0 += 4 * 256) {
+        float wv[4][8];  // four pieces of the row asked for before any is used
+#pragma unroll
+        for (int p = 0; p < 4; ++p)
+          if (d0 + 256 * p < dim) rows_load8(wr + d0 + 256 * p, wv[p]);
+#pragma unroll
+        for (int p = 0; p < 4; ++p)
+          if (d0 + 256 * p < dim) {
+            float xv[8];
+            rows_load8(xs + d0 + 256 * p, xv);
+            a = fmaf(xv[0], wv[p][0], a), b = fmaf(xv[1], wv[p][1], b), c = fmaf(xv[2], wv[p][2], c), d4 = fmaf(xv[3], wv[p][3], d4);
+            a = fmaf(xv[4], wv[p][4], a), b = fmaf(xv[5], wv[p][5], b), c = fmaf(xv[6], wv[p][6], c), d4 = fmaf(xv[7], wv[p][7], d4);
+          }
+      }
+    } else {
+      int d = lane;
+      for (; d + 96 < dim; d += 128) {
+        a = fmaf(xs[d], to_f32(wr[d]), a);
+        b = fmaf(xs[d + 32], to_f32(wr[d + 32]), b);
+        c = fmaf(xs[d + 64], to_f32(wr[d + 64]), c);
+        d4 = fmaf(xs[d + 96], to_f32(wr[d + 96]), d4);
+      }
+      for (; d < dim; d += 32) a = fmaf(xs[d], to_f32(wr[d]), a);
+    }
+    a = warp_sum((a + b) + (c + d4));
+    if (lane == 0) logit[e] = a;
+  }
+  __syncthreads();
+  if (warp == 0)
+    route_choose(logit, logit + experts, expert + (size_t)t * top, weight + (size_t)t * top, experts, top, mode, correction,
+                 route_scale, groups, keep);
+}
+
+__global__ void __launch_bounds__(32 * CHOOSE_WARPS) route_choose_kernel(const float* logits, int* expert, float* weight, int n_tokens,
+                                                                         int experts, int top, int mode, const float* correction,
+                                                                         float route_scale, int groups, int keep) {
+  extern __shared__ float sm[];  // a warp: `experts` logits, `experts` scores, `groups` scores
+  pdl_launch_dependents();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * CHOOSE_WARPS + warp;
+  if (t >= n_tokens) return;
+  float* logit = sm + (size_t)warp * (2 * experts + groups);
+  for (int e = lane; e < experts; e += 32) logit[e] = logits[(size_t)t * experts + e];
+  __syncwarp();
+  route_choose(logit, logit + experts, expert + (size_t)t * top, weight + (size_t)t * top, experts, top, mode, correction,
+               route_scale, groups, keep);
 }
 
 // One block: counts every expert's pairs (in shared memory), then offsets [experts + 1], tile_first [experts + 1]
@@ -447,7 +508,7 @@ __global__ void __launch_bounds__(128) route_scatter_kernel(const T* __restrict_
                                                             const int* __restrict__ offsets, int* __restrict__ placed,
                                                             int* __restrict__ row_of_pair, int* __restrict__ group_of_row,
                                                             T* __restrict__ xs, int dim, int top, int experts, int n_pairs,
-                                                            int weighted) {
+                                                            int weighted, int vec) {
   __shared__ int where;
   pdl_launch_dependents();
   pdl_wait();
@@ -465,7 +526,17 @@ __global__ void __launch_bounds__(128) route_scatter_kernel(const T* __restrict_
   const float wgt = weighted ? ld_fresh(weight + p) : 1.f;
   const T* src = x + (size_t)(p / top) * dim;
   T* dst = xs + (size_t)row * dim;
-  if (weighted)
+  if (vec) {
+    for (int d = 8 * threadIdx.x; d < dim; d += 8 * blockDim.x) {
+      float v[8];
+      rows_load8(src + d, v);
+      if (weighted) {
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v[k] *= wgt;
+      }
+      rows_store8(dst + d, v);
+    }
+  } else if (weighted)
     for (int d = threadIdx.x; d < dim; d += blockDim.x) dst[d] = from_f32<T>(wgt * to_f32(src[d]));
   else
     for (int d = threadIdx.x; d < dim; d += blockDim.x) dst[d] = src[d];
@@ -474,7 +545,7 @@ __global__ void __launch_bounds__(128) route_scatter_kernel(const T* __restrict_
 template <typename T>
 __global__ void __launch_bounds__(256) route_gather_kernel(const T* __restrict__ ys, const int* __restrict__ row_of_pair,
                                                            T* __restrict__ out, int dim, int top, int n_pairs,
-                                                           const float* weight) {
+                                                           const float* weight, int vec) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ int rows_of_token[];  // then, as floats, the pairs' weights
@@ -485,6 +556,22 @@ __global__ void __launch_bounds__(256) route_gather_kernel(const T* __restrict__
     weight_of_token[k] = weight ? ld_fresh(weight + (size_t)t * top + k) : 1.f;
   }
   __syncthreads();
+  if (vec) {
+    for (int d = 8 * threadIdx.x; d < dim; d += 8 * blockDim.x) {
+      float a[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+      for (int k = 0; k < top; ++k) {
+        const int row = rows_of_token[k];
+        if (!FMS_IN(row, n_pairs)) continue;
+        float v[8];
+        rows_load8(ys + (size_t)row * dim + d, v);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) a[e] = fmaf(weight_of_token[k], v[e], a[e]);
+      }
+      rows_store8(out + (size_t)t * dim + d, a);
+    }
+    return;
+  }
   for (int d = threadIdx.x; d < dim; d += blockDim.x) {
     float a = 0.f;
     for (int k = 0; k < top; ++k) {
@@ -553,22 +640,31 @@ FMS_API int fms_grouped_linear(const void* x, const void* w, void* y, int dtype,
 // the rows of xs are the tokens' as they are and fms_route_gather takes the weights.  mode 2: scores sigmoid(logit), the
 // choice by score + correction among the experts of the `keep` best of `groups` equal groups of neighbours (a group's
 // score: the sum of its two largest choice scores), weights the chosen scores times route_scale; rows as in mode 1.
+// logits: [n_tokens, experts] float32 = x . router^T where the caller has them already, else null.
 FMS_API int fms_route(const void* x, int dtype, const void* router, int router_dtype, int* expert, float* weight, int* counts,
                       int* offsets, int* tile_first, int* row_of_pair, int* group_of_row, void* xs, int n_tokens, int dim,
                       int experts, int top, int mode, const float* correction, float route_scale, int groups, int keep,
-                      cudaStream_t stream) {
+                      const float* logits, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (dim <= 0 || experts <= 0 || top <= 0 || top > experts) return fms_fail("route: dim %d, experts %d, top %d", dim, experts, top);
   if (mode < 0 || mode > 2) return fms_fail("route: mode %d", mode);
   if (groups <= 0 || experts % groups || keep <= 0 || keep > groups || (long)keep * (experts / groups) < top)
     return fms_fail("route: %d experts in %d groups of which %d stay, top %d", experts, groups, keep, top);
-  const size_t smem = ((size_t)dim + 2 * (size_t)experts + (size_t)groups) * sizeof(float);
-  if (smem > 200 * 1024) return fms_fail("route: rows of %d values and %d experts do not fit shared memory", dim, experts);
-  FMS_DISPATCH_DTYPE(dtype, T, FMS_DISPATCH_DTYPE(router_dtype, TW, {
-    if (smem > 48 * 1024) cudaFuncSetAttribute(route_kernel<T, TW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    fms_launch(route_kernel<T, TW>, dim3(n_tokens), dim3(32 * ROUTE_WARPS), smem, stream, (const T*)x, (const TW*)router, expert, weight,
-               dim, experts, top, mode, correction, route_scale, groups, keep);
-  }));
+  const int vec = dim % 8 == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)router & 15) == 0 && ((uintptr_t)xs & 15) == 0 ? 1 : 0;
+  const size_t choice = (2 * (size_t)experts + (size_t)groups) * sizeof(float);
+  if (logits != nullptr) {
+    if (CHOOSE_WARPS * choice > 48 * 1024) return fms_fail("route: %d experts in %d groups do not fit shared memory", experts, groups);
+    fms_launch(route_choose_kernel, dim3((n_tokens + CHOOSE_WARPS - 1) / CHOOSE_WARPS), dim3(32 * CHOOSE_WARPS), CHOOSE_WARPS * choice,
+               stream, logits, expert, weight, n_tokens, experts, top, mode, correction, route_scale, groups, keep);
+  } else {
+    const size_t smem = (size_t)dim * sizeof(float) + choice;
+    if (smem > 200 * 1024) return fms_fail("route: rows of %d values and %d experts do not fit shared memory", dim, experts);
+    FMS_DISPATCH_DTYPE(dtype, T, FMS_DISPATCH_DTYPE(router_dtype, TW, {
+      if (smem > 48 * 1024) cudaFuncSetAttribute(route_kernel<T, TW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      fms_launch(route_kernel<T, TW>, dim3(n_tokens), dim3(32 * ROUTE_WARPS), smem, stream, (const T*)x, (const TW*)router, expert,
+                 weight, dim, experts, top, mode, correction, route_scale, groups, keep, vec);
+    }));
+  }
   if (fms_launch_status("route")) return 1;
   const int n_pairs = n_tokens * top;
   fms_launch(route_offsets_kernel, dim3(1), dim3(256), sizeof(int) * experts, stream, (const int*)expert, n_pairs, counts,
@@ -577,7 +673,7 @@ FMS_API int fms_route(const void* x, int dtype, const void* router, int router_d
   FMS_DISPATCH_DTYPE(dtype, T,
                      fms_launch(route_scatter_kernel<T>, dim3(n_pairs), dim3(128), 0, stream, (const T*)x, (const int*)expert,
                                 (const float*)weight, (const int*)offsets, counts, row_of_pair, group_of_row, (T*)xs, dim,
-                                top, experts, n_pairs, mode == 0 ? 1 : 0));
+                                top, experts, n_pairs, mode == 0 ? 1 : 0, vec));
   return fms_launch_status("route (scatter)");
 }
 
@@ -643,6 +739,7 @@ FMS_API int fms_route_gather(const void* ys, int dtype, const int* row_of_pair, 
   if (n_tokens <= 0) return 0;
   FMS_DISPATCH_DTYPE(dtype, T,
                      fms_launch(route_gather_kernel<T>, dim3(n_tokens), dim3(256), 2 * sizeof(int) * top, stream, (const T*)ys, row_of_pair,
-                                (T*)out, dim, top, n_tokens * top, weight));
+                                (T*)out, dim, top, n_tokens * top, weight,
+                                dim % 8 == 0 && ((uintptr_t)ys & 15) == 0 && ((uintptr_t)out & 15) == 0 ? 1 : 0));
   return fms_launch_status("route_gather");
 }

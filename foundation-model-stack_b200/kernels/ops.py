@@ -44,6 +44,8 @@ _SIGNATURES = {
     "fms_rotary_table": [_P, _P, _P, _P, _I, _I, _P],
     "fms_gemm_f32": [_P, _P, _P, _P, _I, _I, _I, _P],
     "fms_linear_bf16_skinny": [_P, _P, _P, _P, _I, _I, _I, _I, _P],
+    "fms_token_gate_bf16_skinny": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
+    "fms_grouped_bf16_skinny": [_P, _P, _P, _P, _I, _I, _I, _I, _P],
     "fms_glu_bf16_skinny": [_P, _P, _P, _P, _I, _I, _I, _I, _P],
     "fms_qkv_rope_store_bf16_skinny": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P,
                                        _I, _I, _I, _P],
@@ -59,7 +61,7 @@ _SIGNATURES = {
     "fms_normed_add_rmsnorm": [_P, _P, _I, _P, _F, _F, _P, _F, _F, _I, _P, _I, _P, _I, _I, _I, _P],
     "fms_mingru_scan": [_P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _P, _P, _I, _P, _P],
     "fms_grouped_linear": [_P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _L, _L, _L, _L, _I, _F, _F, _I, _P],
-    "fms_route": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _F, _I, _I, _P],
+    "fms_route": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _F, _I, _I, _P, _P],
     "fms_route_gather": [_P, _I, _P, _P, _I, _I, _I, _P, _P],
     "fms_relu_squared": [_P, _I, _L, _P],
     "fms_gated_clamped": [_P, _P, _I, _I, _I, _F, _F, _P],
@@ -516,6 +518,18 @@ def gated_activation(gate_up: torch.Tensor, activation: int) -> torch.Tensor:
     return out
 
 
+def token_gated_linear(x: torch.Tensor, weight: torch.Tensor, table: torch.Tensor, tokens: torch.Tensor,
+                       activation: int) -> torch.Tensor:
+    """act(x weight^T) * table[tokens]: one kernel for a few bfloat16 rows, else the product and ``token_gate``."""
+    if (x.dtype == weight.dtype == table.dtype == torch.bfloat16 and x.shape[0] <= SKINNY_ROWS and weight.shape[1] % 8 == 0
+            and activation <= 3 and table.shape[1] == weight.shape[0]):
+        y = torch.empty((x.shape[0], weight.shape[0]), dtype=x.dtype, device=x.device)
+        _call("gemm_bf16_skinny", "fms_token_gate_bf16_skinny", _ptr(x), _ptr(weight), _ptr(table), _ptr(tokens), _ptr(y),
+              x.shape[0], weight.shape[0], weight.shape[1], table.shape[0], int(activation), _stream())
+        return y
+    return token_gate(linear(x, weight), table, tokens, activation)
+
+
 def token_gate(z: torch.Tensor, table: torch.Tensor, tokens: torch.Tensor, activation: int) -> torch.Tensor:
     """act(z[t]) * table[tokens[t]]: rows of a table, one a token, gated by ``z`` [tokens, dim]."""
     n, dim = z.shape
@@ -943,6 +957,7 @@ def gated_group_rmsnorm(x: torch.Tensor, gate: Optional[torch.Tensor], gate_offs
 
 
 # ---- groups of rows, each with a matrix of its own ---------------------------------------------------
+ROUTE_FEW_ROWS = 64  # rows of a step up to which the routing kernel makes the router's product itself
 GROUPED_FEW_ROWS = 32  # rows of a step up to which the grouped products walk each group's rows (a decode step)
 # FMS_B200_GROUPED_LIBRARY=0: the own float32-sum kernel for the ragged products of many bfloat16 rows too
 USE_LIBRARY_GROUPED = os.environ.get("FMS_B200_GROUPED_LIBRARY", "1") != "0" and hasattr(torch.nn.functional, "grouped_mm")
@@ -1006,10 +1021,15 @@ def route(x: torch.Tensor, router: torch.Tensor, top: int, mode: int = ROUTE_SIG
     r.tile_first = ints[o + 2 * (experts + 1): o + 3 * (experts + 1)]
     r.weight = torch.empty((n, top), dtype=torch.float32, device=dev)
     r.rows = torch.empty((n * top, dim), dtype=x.dtype, device=dev)
+    # many bfloat16 rows: the logits from the library's product with float32 results (bfloat16 factors are exact in it)
+    logits = None
+    if x.dtype == router.dtype == torch.bfloat16 and n > ROUTE_FEW_ROWS and 8 * 4 * (2 * experts + groups) <= 48 * 1024:
+        _ptr(x), _ptr(router)
+        logits = torch.mm(x, router.t(), out_dtype=torch.float32)
     _call("grouped", "fms_route", _ptr(x), _code(x.dtype), _ptr(router), _code(router.dtype), _ptr(r.expert),
           _ptr(r.weight), _ptr(counts), _ptr(r.offsets), _ptr(r.tile_first), _ptr(r.row_of_pair), _ptr(r.group_of_row),
           _ptr(r.rows), n, dim, experts, top, int(mode), _ptr(correction), float(route_scale), int(groups), int(keep),
-          _stream())
+          _ptr(logits), _stream())
     global launches
     launches += 2
     return r
@@ -1024,8 +1044,8 @@ def routed_linear(rows: torch.Tensor, weight: torch.Tensor, routing: Routing, gl
     n_out = weight.shape[1] // (2 if glu else 1)
     if weight.dtype != rows.dtype or weight.shape[0] != routing.experts or weight.shape[2] != k:
         raise KernelError(f"routed_linear: rows {rows.dtype} {tuple(rows.shape)}, weight {weight.dtype} {tuple(weight.shape)}")
-    if (USE_LIBRARY_GROUPED and rows.dtype == torch.bfloat16 and n > GROUPED_FEW_ROWS and k % 8 == 0
-            and weight.shape[1] % 8 == 0):
+    if (USE_LIBRARY_GROUPED and rows.dtype == torch.bfloat16 and n > max(GROUPED_FEW_ROWS, SKINNY_ROWS * routing.top)
+            and k % 8 == 0 and weight.shape[1] % 8 == 0):
         # many bfloat16 rows: the library's grouped product (it takes the groups' ends from the device, as the
         # own kernels do), as the plain products of many rows take the library's; the gated unit is a kernel after it
         _ptr(rows), _ptr(weight)
@@ -1041,6 +1061,11 @@ def routed_linear(rows: torch.Tensor, weight: torch.Tensor, routing: Routing, gl
               _stream())
         return out
     y = torch.empty((n, n_out), dtype=rows.dtype, device=rows.device)
+    if rows.dtype == torch.bfloat16 and n <= SKINNY_ROWS * routing.top and k % 8 == 0 and (silu or not glu):
+        # up to eight tokens, so up to eight rows an expert: the weight-streaming kernel, a block per group and run of rows
+        _call("gemm_bf16_skinny", "fms_grouped_bf16_skinny", _ptr(rows), _ptr(weight), _ptr(y), _ptr(routing.offsets),
+              routing.experts, n_out, k, 3 if glu else (2 if relu_squared else 0), _stream())
+        return y
     _call("grouped", "fms_grouped_linear", _ptr(rows), _ptr(weight), _ptr(y), _code(rows.dtype), _ptr(routing.offsets),
           _ptr(routing.tile_first), _ptr(routing.group_of_row), routing.experts, n, n_out, k, k, 0, n_out, 0,
           (3 if silu else 1) if glu else (2 if relu_squared else 0), float(limit), float(alpha), 1 if n <= GROUPED_FEW_ROWS else 0, _stream())

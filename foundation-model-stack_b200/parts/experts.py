@@ -29,6 +29,8 @@ Further options, each of which leaves the above as it is when absent:
 """
 from __future__ import annotations
 
+import torch
+
 from ..config.specs import FeedForwardSpec
 from ..kernels import ops
 from .base import Part
@@ -102,7 +104,7 @@ class RoutedExperts(Part):
         return ops.route_gather(ops.routed_linear(hidden, self.tensor("down"), routing), routing)
 
     def kernel_libraries(self, dtype):
-        return ["grouped", "elementwise"]
+        return ["grouped", "elementwise"] + (["gemm_bf16_skinny"] if dtype == torch.bfloat16 else [])
 
 
 register_feed_forward("routed_experts", RoutedExperts)

@@ -39,7 +39,7 @@ class TokenSide(Part):
             x = residual
         else:
             x = ops.normed_add_norm(residual, parts, None, None, dtype)
-        g = ops.token_gate(self.gate.forward(x), self.tensor("table"), batch.tokens, self.activation)
+        g = ops.token_gated_linear(x, self.gate.tensor("weight"), self.tensor("table"), batch.tokens, self.activation)
         return NormedDelta(self.proj.forward(g), self.norm)
 
     def kernel_libraries(self, dtype):
