@@ -56,7 +56,7 @@ class MixerSpec:
 
 @dataclasses.dataclass(frozen=True)
 class FeedForwardSpec:
-    """``kind == "glu"``: down(act(gate(x)) * up(x)) with fused [gate; up] rows."""
+    """``kind == "glu"``: down(act(gate(x)) * up(x)) with fused [gate; up] rows; ``"mlp"``: down(act(up(x)))."""
 
     kind: str
     dim: int
@@ -88,7 +88,8 @@ class BlockSpec:
     normed once more before it is added, x += norm1b(mixer(norm1(x))); x += norm2b(feed_forward(norm2(x))); the two
     further norms are ``mixer_post_norm`` and ``feed_forward_post_norm``, and a layer without a feed-forward
     (``feed_forward is None``) ends after its mixer.  ``arrangement == "parallel_joint"``: both sublayers read one norm,
-    x += mixer(norm1(x)) + feed_forward(norm1(x)), through one joint projection, and ``token_side`` (optional) follows.  The names are those under which the layer's
+    x += mixer(norm1(x)) + feed_forward(norm1(x)), through one joint projection, and ``token_side`` (optional) follows.  ``arrangement == "hyper_connected"``: pre-norm
+    sublayers between ``streams`` (in ``options`` and in the ``DecoderSpec``) residual streams a token.  The names are those under which the layer's
     parts appear in weight names (``ln``, ``attn``, ``ff_ln``, ``ff_sub_layer`` for Llama); ``post_names`` those of
     the two further norms."""
 
@@ -147,6 +148,8 @@ class DecoderSpec:
     names: Tuple[str, str, str, str] = ("base_model.embedding", "base_model.layers", "base_model.dec_norm", "head")
     embedding_scale: float = 1.0  # the embedded rows are multiplied by it as they enter the residual stream
     logit_scale: float = 1.0  # the logits are multiplied by it
+    logit_softcap: float = 0.0  # then, where it is positive, z becomes softcap * tanh(z / softcap)
+    streams: int = 0  # residual streams a token of layers that mix several (``"hyper_connected"``); 0: the one stream
     embedding: EmbeddingSpec = EmbeddingSpec()
 
     def __post_init__(self):

@@ -1411,3 +1411,245 @@ FMS_API int fms_sigmoid_gate(const void* o, const void* gate, int gate_stride, v
   }
   return fms_launch_status("sigmoid_gate");
 }
+
+// ---------------------------------------------------------------------------------------------------
+// several residual streams a token (hyper-connections): what the sublayer before left pending goes into all of them, and
+// the next sublayer's input is mixed from them and normed, in one pass over the token's rows
+//   new_t = sum_s mix[s][t] old_s + w_out[t] * delta        (no delta: new_t = old_t and nothing is written)
+//   u     = sum_t w_in[t] new_t
+//   out   = u / sqrt(mean(u^2) + eps) * gain                 (no gain: out = u)
+// src: [rows, src_streams, dim] float32, src_streams the number of streams, or 1 where all of them still are the same row
+// (a token's embedding); dst [rows, streams, dim] (may be src) or null: nothing is written.  `on`: mix [streams, streams],
+// then w_out [streams].  rows: the tokens to compute (no dst then).  A block a token; four neighbouring columns a thread and
+// NCHUNK such runs; a thread reads every stream's values of its columns before it writes any.
+// ---------------------------------------------------------------------------------------------------
+template <typename T, int MAXS, int NCHUNK>
+__global__ void stream_mix_norm_kernel(const float* src, int src_streams, float* dst, const T* delta, const float* on,
+                                       const float* w_in, const float* gain, float eps, T* out, const int* rows, int dim,
+                                       int streams, int residual_rows) {
+  __shared__ float scratch[33];
+  pdl_launch_dependents();
+  float mix[MAXS][MAXS], w_out[MAXS], win[MAXS];  // weights: read ahead of the wait
+#pragma unroll
+  for (int t = 0; t < MAXS; ++t) {
+    win[t] = t < streams ? w_in[t] : 0.f;
+    w_out[t] = delta && t < streams ? on[streams * streams + t] : 0.f;
+#pragma unroll
+    for (int s = 0; s < MAXS; ++s) mix[s][t] = delta && s < streams && t < streams ? on[s * streams + t] : 0.f;
+  }
+  pdl_wait();
+  const int r = blockIdx.x;
+  const int tok = rows ? rows[r] : r;
+  if (!FMS_IN(tok, residual_rows)) return;  // the whole block alike
+  const float* from = src + (size_t)tok * src_streams * dim;
+  float* to = dst ? dst + (size_t)tok * streams * dim : nullptr;
+  const T* del = delta ? delta + (size_t)tok * dim : nullptr;
+  float u[NCHUNK][4];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < NCHUNK; ++j) {
+    const int d = (threadIdx.x + j * blockDim.x) * 4;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) u[j][k] = 0.f;
+    if (d >= dim) continue;
+    float x[MAXS][4], y[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int s = 0; s < MAXS; ++s)
+      if (s < streams) ldv4(from + (size_t)(src_streams == 1 ? 0 : s) * dim + d, x[s]);
+    if (del) ldv4(del + d, y);
+#pragma unroll
+    for (int t = 0; t < MAXS; ++t) {
+      if (t < streams) {
+        float n[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) n[k] = del ? w_out[t] * y[k] : x[t][k];
+        if (del) {
+#pragma unroll
+          for (int s = 0; s < MAXS; ++s)
+            if (s < streams) {
+#pragma unroll
+              for (int k = 0; k < 4; ++k) n[k] = fmaf(mix[s][t], x[s][k], n[k]);
+            }
+        }
+        if (to) stv4(to + (size_t)t * dim + d, n);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) u[j][k] = fmaf(win[t], n[k], u[j][k]);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k) ss = fmaf(u[j][k], u[j][k], ss);
+  }
+  const float inv = gain ? 1.f / sqrtf(block_sum(ss, scratch) / (float)dim + eps) : 1.f;
+  T* o = out + (size_t)r * dim;
+#pragma unroll
+  for (int j = 0; j < NCHUNK; ++j) {
+    const int d = (threadIdx.x + j * blockDim.x) * 4;
+    if (d >= dim) continue;
+    float g[4] = {1.f, 1.f, 1.f, 1.f};
+    if (gain) ldv4(gain + d, g);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) g[k] *= u[j][k] * inv;
+    stv4(o + d, g);
+  }
+}
+
+// The same for any width and up to MAX_STREAMS streams: a column a thread at a time, the mixed row in shared memory.
+constexpr int MAX_STREAMS = 16;
+
+template <typename T>
+__global__ void stream_mix_norm_any_kernel(const float* src, int src_streams, float* dst, const T* delta, const float* on,
+                                           const float* w_in, const float* gain, float eps, T* out, const int* rows, int dim,
+                                           int streams, int residual_rows) {
+  extern __shared__ float u[];  // [dim]
+  __shared__ float scratch[33];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int r = blockIdx.x;
+  const int tok = rows ? rows[r] : r;
+  if (!FMS_IN(tok, residual_rows)) return;  // the whole block alike
+  const float* from = src + (size_t)tok * src_streams * dim;
+  float* to = dst ? dst + (size_t)tok * streams * dim : nullptr;
+  const T* del = delta ? delta + (size_t)tok * dim : nullptr;
+  float ss = 0.f;
+  for (int d = threadIdx.x; d < dim; d += blockDim.x) {
+    float x[MAX_STREAMS];
+#pragma unroll
+    for (int s = 0; s < MAX_STREAMS; ++s) x[s] = s < streams ? from[(size_t)(src_streams == 1 ? 0 : s) * dim + d] : 0.f;
+    float sum = 0.f;
+    if (del) {
+      const float y = to_f32(del[d]);
+      for (int t = 0; t < streams; ++t) {
+        float n = on[streams * streams + t] * y;
+#pragma unroll
+        for (int s = 0; s < MAX_STREAMS; ++s)
+          if (s < streams) n = fmaf(on[s * streams + t], x[s], n);
+        if (to) to[(size_t)t * dim + d] = n;
+        sum = fmaf(w_in[t], n, sum);
+      }
+    } else {
+#pragma unroll
+      for (int s = 0; s < MAX_STREAMS; ++s)
+        if (s < streams) sum = fmaf(w_in[s], x[s], sum);
+    }
+    u[d] = sum;
+    ss = fmaf(sum, sum, ss);
+  }
+  const float inv = gain ? 1.f / sqrtf(block_sum(ss, scratch) / (float)dim + eps) : 1.f;
+  for (int d = threadIdx.x; d < dim; d += blockDim.x)  // a thread's own columns
+    out[(size_t)r * dim + d] = from_f32<T>(u[d] * inv * (gain ? gain[d] : 1.f));
+}
+
+FMS_API int fms_stream_mix_norm(const float* src, int src_streams, float* dst, const void* delta, const float* on,
+                                const float* w_in, const float* gain, float eps, void* out, int dtype, const int* rows,
+                                int n_rows, int dim, int streams, int residual_rows, cudaStream_t stream) {
+  if (n_rows <= 0) return 0;
+  if (streams < 1 || streams > MAX_STREAMS || (src_streams != 1 && src_streams != streams) || dim <= 0 || dim > 48 * 1024)
+    return fms_fail("stream_mix_norm: %d streams (up to %d) from %d, width %d (up to 49152)", streams, MAX_STREAMS, src_streams, dim);
+  if (!w_in || !out || (delta && !on) || (dst && !delta) || (dst && rows) || (dst == src && src_streams != streams))
+    return fms_fail("stream_mix_norm: weights, an output and, where the streams are written, what goes into them");
+  const size_t item = dtype == FMS_BF16 ? 2 : 4;
+  const bool four = dim % 4 == 0 && (uintptr_t)src % 16 == 0 && (uintptr_t)dst % 16 == 0 && (uintptr_t)gain % 16 == 0 &&
+                    (uintptr_t)delta % (4 * item) == 0 && (uintptr_t)out % (4 * item) == 0;
+  if (!four || streams > 4 || dim > 4 * 4 * 1024) {
+    const size_t smem = (size_t)dim * sizeof(float);
+    FMS_DISPATCH_DTYPE(dtype, T, {
+      if (smem > 47 * 1024)
+        cudaFuncSetAttribute(stream_mix_norm_any_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      fms_launch(stream_mix_norm_any_kernel<T>, dim3(n_rows), dim3(dim >= 1024 ? 512 : 128), smem, stream, src, src_streams, dst,
+                 (const T*)delta, on, w_in, gain, eps, (T*)out, rows, dim, streams, residual_rows);
+    });
+    return fms_launch_status("stream_mix_norm");
+  }
+  const int runs = dim / 4;
+  int threads = 128;
+  // few rows: a run a thread, the shortest chain a row can have; many: two, where more blocks hide one another's waits
+  while (threads < 1024 && threads * (n_rows <= 148 ? 1 : 2) < runs) threads *= 2;
+  const int nchunk = (runs + threads - 1) / threads;
+#define FMS_SMN(MAXS, NCHUNK)                                                                                               \
+  FMS_DISPATCH_DTYPE(dtype, T, fms_launch(stream_mix_norm_kernel<T, MAXS, NCHUNK>, dim3(n_rows), dim3(threads), 0, stream,  \
+                                          src, src_streams, dst, (const T*)delta, on, w_in, gain, eps, (T*)out, rows, dim,  \
+                                          streams, residual_rows))
+  if (streams <= 2) {
+    if (nchunk <= 1) FMS_SMN(2, 1);
+    else if (nchunk <= 2) FMS_SMN(2, 2);
+    else FMS_SMN(2, 4);
+  } else {
+    if (nchunk <= 1) FMS_SMN(4, 1);
+    else if (nchunk <= 2) FMS_SMN(4, 2);
+    else FMS_SMN(4, 4);
+  }
+#undef FMS_SMN
+  return fms_launch_status("stream_mix_norm");
+}
+
+// ---------------------------------------------------------------------------------------------------
+// an activation of every value, in place (the hidden values of an ungated feed-forward after a library product)
+// ---------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void activation_kernel(T* y, int act, size_t total) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x)
+    y[i] = from_f32<T>(activate(to_f32(y[i]), act));
+}
+
+__global__ void activation_vec_kernel(__nv_bfloat16* y, int act, size_t total8) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < total8; i += (size_t)gridDim.x * blockDim.x) {
+    float v[8];
+    embed_load8(y + 8 * i, v);
+    uint32_t o[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const __nv_bfloat162 b = __floats2bfloat162_rn(activate(v[2 * k], act), activate(v[2 * k + 1], act));
+      o[k] = *reinterpret_cast<const uint32_t*>(&b);
+    }
+    *reinterpret_cast<uint4*>(y + 8 * i) = make_uint4(o[0], o[1], o[2], o[3]);
+  }
+}
+
+FMS_API int fms_activation(void* y, int dtype, int act, long total, cudaStream_t stream) {
+  if (total <= 0) return 0;
+  if (act < 0 || act > 4) return fms_fail("activation: %d", act);
+  if (dtype == FMS_BF16 && total % 8 == 0 && ((uintptr_t)y & 15) == 0) {
+    const long total8 = total / 8;
+    const int blocks = (int)((total8 + 255) / 256 < 148 * 32 ? (total8 + 255) / 256 : 148 * 32);
+    fms_launch(activation_vec_kernel, dim3(blocks), dim3(256), 0, stream, (__nv_bfloat16*)y, act, (size_t)total8);
+    return fms_launch_status("activation");
+  }
+  const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
+  FMS_DISPATCH_DTYPE(dtype, T, fms_launch(activation_kernel<T>, dim3(blocks), dim3(256), 0, stream, (T*)y, act, (size_t)total));
+  return fms_launch_status("activation");
+}
+
+// ---------------------------------------------------------------------------------------------------
+// logits, in place: z * scale, then, with cap > 0, cap * tanh(. / cap)
+// ---------------------------------------------------------------------------------------------------
+template <int VEC>
+__global__ void scale_cap_kernel(float* z, float scale, float cap, size_t runs) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < runs; i += (size_t)gridDim.x * blockDim.x) {
+    float v[4] = {0.f, 0.f, 0.f, 0.f};
+    if constexpr (VEC == 4) ldv4(z + 4 * i, v);
+    else v[0] = z[i];
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) {
+      v[k] *= scale;
+      if (cap > 0.f) v[k] = cap * tanhf(v[k] / cap);
+    }
+    if constexpr (VEC == 4) stv4(z + 4 * i, v);
+    else z[i] = v[0];
+  }
+}
+
+FMS_API int fms_scale_cap(float* z, float scale, float cap, long total, cudaStream_t stream) {
+  if (total <= 0) return 0;
+  const bool four = total % 4 == 0 && (uintptr_t)z % 16 == 0;
+  const long runs = four ? total / 4 : total;
+  const int blocks = (int)((runs + 255) / 256 < 148 * 8 ? (runs + 255) / 256 : 148 * 8);
+  if (four) fms_launch(scale_cap_kernel<4>, dim3(blocks), dim3(256), 0, stream, z, scale, cap, (size_t)runs);
+  else fms_launch(scale_cap_kernel<1>, dim3(blocks), dim3(256), 0, stream, z, scale, cap, (size_t)runs);
+  return fms_launch_status("scale_cap");
+}

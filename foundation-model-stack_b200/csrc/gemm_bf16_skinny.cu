@@ -47,13 +47,15 @@ struct RopeArgs {
   int n_seqs, table_rows, pool_blocks;  // extents of slots, of the table and of the cache, for the bounds-checked build
 };
 
-// What the ROWS16 epilogue does beyond the product: nothing, or y = act(v) * table[tokens[m]] (table set), or the square of
-// relu (squares).  offsets: GROUPED only.
+// What the ROWS16 epilogue does beyond the product: nothing, or y = act(v) * table[tokens[m]] (table set), or what `unit`
+// says: the square of relu, act(v), or v * scale, capped by cap * tanh(. / cap) where cap > 0.  offsets: GROUPED only.
+enum Unit { UNIT_NONE = 0, UNIT_SQUARES = 1, UNIT_ACT = 2, UNIT_CAP = 3 };
 struct RowArgs {
   const __nv_bfloat16* table;  // [vocab, N]
   const int* tokens;           // [M]
-  int vocab, squares;
+  int vocab, unit;
   const int* offsets;          // [groups + 1]
+  float scale, cap;
 };
 
 __device__ __forceinline__ void mma_bf16(float* d, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
@@ -282,9 +284,14 @@ __global__ void __launch_bounds__(THREADS) linear_skinny_kernel(const __nv_bfloa
         if (extra.table) {
           const int tok = __ldcg(extra.tokens + m);  // a token outside the vocabulary: the embedding has set the flag
           v = tok >= 0 && tok < extra.vocab ? activate(v, act) * __bfloat162float(extra.table[(size_t)tok * N + row]) : 0.f;
-        } else if (extra.squares) {
+        } else if (extra.unit == UNIT_SQUARES) {
           v = fmaxf(v, 0.f);
           v *= v;
+        } else if (extra.unit == UNIT_ACT) {
+          v = activate(v, act);
+        } else if (extra.unit == UNIT_CAP) {
+          v *= extra.scale;
+          if (extra.cap > 0.f) v = extra.cap * tanhf(v / extra.cap);
         }
         if (FMS_IN((size_t)m * N + row, (size_t)M * N)) y[(size_t)m * N + row] = from_f32<TOut>(v);
       }
@@ -338,6 +345,27 @@ FMS_API int fms_linear_bf16_skinny(const void* x, const void* w, const void* bia
   return launch<1, 2, ROWS16>(x, w, bias, y, out_dtype, M, N, K, 0, 0, stream);
 }
 
+// y [M, N] bfloat16 = act(x w[N, K]^T + bias): the first product of an ungated feed-forward.
+FMS_API int fms_linear_act_bf16_skinny(const void* x, const void* w, const void* bias, void* y, int M, int N, int K, int act,
+                                       cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (M > 8) return fms_fail("linear_act_bf16_skinny: %d rows, at most 8", M);
+  if (K <= 0 || K % 8 || act < 0 || act > 3) return fms_fail("linear_act_bf16_skinny: K %d, activation %d", K, act);
+  const RowArgs extra{nullptr, nullptr, 0, UNIT_ACT, nullptr, 1.f, 0.f};
+  return launch_typed<1, 1, ROWS16, __nv_bfloat16>(x, w, bias, y, M, N, K, 0, act, stream, RopeArgs{}, extra);
+}
+
+// y [M, N] float32 = x w[N, K]^T * scale, capped where cap > 0: the logits of a decode step.
+FMS_API int fms_linear_cap_bf16_skinny(const void* x, const void* w, void* y, int M, int N, int K, float scale, float cap,
+                                       cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (M > 8) return fms_fail("linear_cap_bf16_skinny: %d rows, at most 8", M);
+  if (K <= 0 || K % 8) return fms_fail("linear_cap_bf16_skinny: K %d must be a positive multiple of 8", K);
+  const RowArgs extra{nullptr, nullptr, 0, UNIT_CAP, nullptr, scale, cap};
+  if (N < 16384) return launch_typed<1, 1, ROWS16, float>(x, w, nullptr, y, M, N, K, 0, 0, stream, RopeArgs{}, extra);
+  return launch_typed<1, 2, ROWS16, float>(x, w, nullptr, y, M, N, K, 0, 0, stream, RopeArgs{}, extra);
+}
+
 // y [M, N] = act(x w[N, K]^T) * table[tokens[m], :]: a small product gated by the tokens' own rows of a table [vocab, N].
 FMS_API int fms_token_gate_bf16_skinny(const void* x, const void* w, const void* table, const int* tokens, void* y, int M, int N,
                                        int K, int vocab, int act, cudaStream_t stream) {
@@ -345,7 +373,7 @@ FMS_API int fms_token_gate_bf16_skinny(const void* x, const void* w, const void*
   if (M > 8) return fms_fail("token_gate_bf16_skinny: %d rows, at most 8", M);
   if (K <= 0 || K % 8 || vocab <= 0 || act < 0 || act > 3 || !table || !tokens)
     return fms_fail("token_gate_bf16_skinny: K %d, vocabulary %d, activation %d", K, vocab, act);
-  const RowArgs extra{(const __nv_bfloat16*)table, tokens, vocab, 0, nullptr};
+  const RowArgs extra{(const __nv_bfloat16*)table, tokens, vocab, UNIT_NONE, nullptr, 1.f, 0.f};
   return launch_typed<1, 1, ROWS16, __nv_bfloat16>(x, w, nullptr, y, M, N, K, 0, act, stream, RopeArgs{}, extra);
 }
 
@@ -356,7 +384,7 @@ FMS_API int fms_grouped_bf16_skinny(const void* x, const void* w, void* y, const
   if (groups <= 0 || N <= 0) return 0;
   if (groups > 65535 || K <= 0 || K % 8 || !offsets || (kind != 0 && kind != 2 && kind != 3))
     return fms_fail("grouped_bf16_skinny: %d groups, K %d, kind %d", groups, K, kind);
-  const RowArgs extra{nullptr, nullptr, 0, kind == 2 ? 1 : 0, offsets};
+  const RowArgs extra{nullptr, nullptr, 0, kind == 2 ? UNIT_SQUARES : UNIT_NONE, offsets, 1.f, 0.f};
   if (kind == 3)
     return launch_typed<1, 2, GLU8, __nv_bfloat16, true>(x, w, nullptr, y, 8, 2 * N, K, N, 0, stream, RopeArgs{}, extra, groups);
   return launch_typed<1, 1, ROWS16, __nv_bfloat16, true>(x, w, nullptr, y, 8, N, K, 0, 0, stream, RopeArgs{}, extra, groups);

@@ -50,6 +50,7 @@ struct Epilogue {
   int glu;            // 1: the first half of the accumulator's columns are gate rows, the second the matching up rows
   int hidden;         // GLU: rows of the gate matrix
   int act;
+  int plain_act;      // plain only, 1: act of every value
   int tile_n;         // accumulator columns of a tile: rows of w per tile (GLU: gate and up together)
   int stages;
   // The fused projection of an attention layer (qkv 1): rows of w are [q heads | k heads | v heads]; q and k are
@@ -109,6 +110,10 @@ __device__ __forceinline__ void store_rows(const Epilogue& ep, uint32_t taddr, i
 #pragma unroll
       for (int jj = 0; jj < 16; ++jj)
         if (col0 + jj < ncols) v[jj] += __bfloat162float(bias[col0 + jj]);
+    }
+    if (ep.plain_act) {
+#pragma unroll
+      for (int jj = 0; jj < 16; ++jj) v[jj] = activate(v[jj], ep.act);
     }
     if (row >= M || col0 >= ncols) continue;  // nothing of these 16 columns lies inside y
     if (ep.qkv) {
@@ -505,6 +510,19 @@ FMS_API int fms_gemm_bf16_tc(const void* x, const void* w, const void* bias, voi
   ep.out = y;
   ep.bias = bias;
   ep.out_f32 = out_dtype == FMS_F32 ? 1 : 0;
+  return launch(x, w, N, ep, M, N, K, error_flag, stream);
+}
+
+// y [M, N] bfloat16 = act(x w[N, K]^T + bias): the first product of an ungated feed-forward.
+FMS_API int fms_linear_act_bf16_tc(const void* x, const void* w, const void* bias, void* y, int M, int N, int K, int act,
+                                   int* error_flag, cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (act < 0 || act > 3) return fms_fail("linear_act_tc: activation %d", act);
+  Epilogue ep = {};
+  ep.out = y;
+  ep.bias = bias;
+  ep.act = act;
+  ep.plain_act = 1;
   return launch(x, w, N, ep, M, N, K, error_flag, stream);
 }
 

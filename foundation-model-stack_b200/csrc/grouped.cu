@@ -309,6 +309,7 @@ __global__ void gated_clamped_vec_kernel(const __nv_bfloat16* gu, __nv_bfloat16*
 constexpr int ROUTE_WARPS = 16, CHOOSE_WARPS = 8;
 
 // What a warp does with one token's logits (in shared memory, `score` behind them: experts + groups values of scratch).
+// Mode 3: the choice is by logit, the weights are the softmax over the chosen logits only, times route_scale.
 __device__ __forceinline__ void route_choose(float* logit, float* score, int* expert, float* weight, int experts, int top, int mode,
                              const float* correction, float route_scale, int groups, int keep) {
   const int lane = threadIdx.x & 31;
@@ -365,7 +366,7 @@ __device__ __forceinline__ void route_choose(float* logit, float* score, int* ex
       __syncwarp();
     }
   }
-  float picked_sum = 0.f;
+  float picked_sum = 0.f, first = 0.f;
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
     int at = 0x7fffffff;
@@ -385,17 +386,20 @@ __device__ __forceinline__ void route_choose(float* logit, float* score, int* ex
         at = oa;
       }
     }
+    if (k == 0) first = best;  // the largest logit: what the exponentials of mode 3 are taken against
     if (at >= experts) at = k;  // every logit was NaN or -inf: any expert, so that nothing below reads outside
     if (lane == 0) {
       expert[k] = at;
-      weight[k] = mode == 1 ? score[at] : (mode == 2 ? score[at] * route_scale : 1.f / (1.f + expf(-best)));
+      weight[k] = mode == 1 ? score[at] : (mode == 2 ? score[at] * route_scale
+                                                     : (mode == 3 ? expf(best - first) : 1.f / (1.f + expf(-best))));
       logit[at] = -INFINITY;
     }
     if (mode == 1) picked_sum += score[at];
+    if (mode == 3) picked_sum += expf(best - first);
     __syncwarp();
   }
-  if (mode == 1 && lane == 0) {
-    const float f = route_scale / (picked_sum + 1e-20f);
+  if ((mode == 1 || mode == 3) && lane == 0) {
+    const float f = mode == 3 ? route_scale / picked_sum : route_scale / (picked_sum + 1e-20f);
     for (int k = 0; k < top; ++k) weight[k] *= f;
   }
 }
@@ -403,7 +407,8 @@ __device__ __forceinline__ void route_choose(float* logit, float* score, int* ex
 template <typename T, typename TW>
 __global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(const T* x, const TW* router, int* expert, float* weight, int dim,
                                                                  int experts, int top, int mode, const float* correction,
-                                                                 float route_scale, int groups, int keep, int vec) {
+                                                                 float route_scale, int groups, int keep, int vec,
+                                                                 const float* bias, float* side) {
   extern __shared__ float sm[];  // dim values of x, `experts` logits, `experts` scores (mode 1, 2), `groups` scores (mode 2)
   float* xs = sm;
   float* logit = sm + dim;
@@ -420,7 +425,7 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(const T* x, con
     for (int d = threadIdx.x; d < dim; d += blockDim.x) xs[d] = to_f32(x[(size_t)t * dim + d]);
   }
   __syncthreads();
-  for (int e = warp; e < experts; e += ROUTE_WARPS) {
+  for (int e = warp; e < experts + (side ? 1 : 0); e += ROUTE_WARPS) {
     const TW* wr = router + (size_t)e * dim;
     float a = 0.f, b = 0.f, c = 0.f, d4 = 0.f;  // four chains: the loads of one do not wait for another's sum
     if (vec) {
@@ -449,7 +454,10 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(const T* x, con
       for (; d < dim; d += 32) a = fmaf(xs[d], to_f32(wr[d]), a);
     }
     a = warp_sum((a + b) + (c + d4));
-    if (lane == 0) logit[e] = a;
+    if (lane == 0) {
+      if (e == experts) side[t] = 1.f / (1.f + expf(-a));  // the row behind the experts': the shared unit's gate
+      else logit[e] = bias ? a + bias[e] : a;
+    }
   }
   __syncthreads();
   if (warp == 0)
@@ -459,14 +467,17 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(const T* x, con
 
 __global__ void __launch_bounds__(32 * CHOOSE_WARPS) route_choose_kernel(const float* logits, int* expert, float* weight, int n_tokens,
                                                                          int experts, int top, int mode, const float* correction,
-                                                                         float route_scale, int groups, int keep) {
+                                                                         float route_scale, int groups, int keep,
+                                                                         const float* bias, float* side) {
   extern __shared__ float sm[];  // a warp: `experts` logits, `experts` scores, `groups` scores
   pdl_launch_dependents();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * CHOOSE_WARPS + warp;
   if (t >= n_tokens) return;
   float* logit = sm + (size_t)warp * (2 * experts + groups);
-  for (int e = lane; e < experts; e += 32) logit[e] = logits[(size_t)t * experts + e];
+  const float* mine = logits + (size_t)t * (experts + (side ? 1 : 0));
+  for (int e = lane; e < experts; e += 32) logit[e] = bias ? mine[e] + bias[e] : mine[e];
+  if (side && lane == 0) side[t] = 1.f / (1.f + expf(-mine[experts]));
   __syncwarp();
   route_choose(logit, logit + experts, expert + (size_t)t * top, weight + (size_t)t * top, experts, top, mode, correction,
                route_scale, groups, keep);
@@ -545,7 +556,8 @@ __global__ void __launch_bounds__(128) route_scatter_kernel(const T* __restrict_
 template <typename T>
 __global__ void __launch_bounds__(256) route_gather_kernel(const T* __restrict__ ys, const int* __restrict__ row_of_pair,
                                                            T* __restrict__ out, int dim, int top, int n_pairs,
-                                                           const float* weight, int vec) {
+                                                           const float* weight, const T* shared, const float* side,
+                                                           int vec) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ int rows_of_token[];  // then, as floats, the pairs' weights
@@ -556,9 +568,16 @@ __global__ void __launch_bounds__(256) route_gather_kernel(const T* __restrict__
     weight_of_token[k] = weight ? ld_fresh(weight + (size_t)t * top + k) : 1.f;
   }
   __syncthreads();
+  const T* every = shared ? shared + (size_t)t * dim : nullptr;
+  const float gate = every && side ? ld_fresh(side + t) : 1.f;
   if (vec) {
     for (int d = 8 * threadIdx.x; d < dim; d += 8 * blockDim.x) {
       float a[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      if (every) {
+        rows_load8(every + d, a);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) a[e] *= gate;
+      }
 #pragma unroll 4
       for (int k = 0; k < top; ++k) {
         const int row = rows_of_token[k];
@@ -573,7 +592,7 @@ __global__ void __launch_bounds__(256) route_gather_kernel(const T* __restrict__
     return;
   }
   for (int d = threadIdx.x; d < dim; d += blockDim.x) {
-    float a = 0.f;
+    float a = every ? gate * to_f32(every[d]) : 0.f;
     for (int k = 0; k < top; ++k) {
       const int row = rows_of_token[k];
       if (FMS_IN(row, n_pairs)) a = fmaf(weight_of_token[k], to_f32(ys[(size_t)row * dim + d]), a);
@@ -640,14 +659,17 @@ FMS_API int fms_grouped_linear(const void* x, const void* w, void* y, int dtype,
 // the rows of xs are the tokens' as they are and fms_route_gather takes the weights.  mode 2: scores sigmoid(logit), the
 // choice by score + correction among the experts of the `keep` best of `groups` equal groups of neighbours (a group's
 // score: the sum of its two largest choice scores), weights the chosen scores times route_scale; rows as in mode 1.
-// logits: [n_tokens, experts] float32 = x . router^T where the caller has them already, else null.
+// mode 3: the choice is by logit, weights the softmax over the chosen logits only, times route_scale; rows as in mode 1.
+// logits: [n_tokens, rows of router] float32 = x . router^T where the caller has them already, else null.
+// bias: [experts] float32 that is added to the logits first, or null.  side: [n_tokens] float32, or null: the router then has
+// a row behind the experts' and side[t] = sigmoid(x[t] . that row), the gate of a unit that every token uses.
 FMS_API int fms_route(const void* x, int dtype, const void* router, int router_dtype, int* expert, float* weight, int* counts,
                       int* offsets, int* tile_first, int* row_of_pair, int* group_of_row, void* xs, int n_tokens, int dim,
                       int experts, int top, int mode, const float* correction, float route_scale, int groups, int keep,
-                      const float* logits, cudaStream_t stream) {
+                      const float* logits, const float* bias, float* side, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (dim <= 0 || experts <= 0 || top <= 0 || top > experts) return fms_fail("route: dim %d, experts %d, top %d", dim, experts, top);
-  if (mode < 0 || mode > 2) return fms_fail("route: mode %d", mode);
+  if (mode < 0 || mode > 3) return fms_fail("route: mode %d", mode);
   if (groups <= 0 || experts % groups || keep <= 0 || keep > groups || (long)keep * (experts / groups) < top)
     return fms_fail("route: %d experts in %d groups of which %d stay, top %d", experts, groups, keep, top);
   const int vec = dim % 8 == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)router & 15) == 0 && ((uintptr_t)xs & 15) == 0 ? 1 : 0;
@@ -655,14 +677,14 @@ FMS_API int fms_route(const void* x, int dtype, const void* router, int router_d
   if (logits != nullptr) {
     if (CHOOSE_WARPS * choice > 48 * 1024) return fms_fail("route: %d experts in %d groups do not fit shared memory", experts, groups);
     fms_launch(route_choose_kernel, dim3((n_tokens + CHOOSE_WARPS - 1) / CHOOSE_WARPS), dim3(32 * CHOOSE_WARPS), CHOOSE_WARPS * choice,
-               stream, logits, expert, weight, n_tokens, experts, top, mode, correction, route_scale, groups, keep);
+               stream, logits, expert, weight, n_tokens, experts, top, mode, correction, route_scale, groups, keep, bias, side);
   } else {
     const size_t smem = (size_t)dim * sizeof(float) + choice;
     if (smem > 200 * 1024) return fms_fail("route: rows of %d values and %d experts do not fit shared memory", dim, experts);
     FMS_DISPATCH_DTYPE(dtype, T, FMS_DISPATCH_DTYPE(router_dtype, TW, {
       if (smem > 48 * 1024) cudaFuncSetAttribute(route_kernel<T, TW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       fms_launch(route_kernel<T, TW>, dim3(n_tokens), dim3(32 * ROUTE_WARPS), smem, stream, (const T*)x, (const TW*)router, expert,
-                 weight, dim, experts, top, mode, correction, route_scale, groups, keep, vec);
+                 weight, dim, experts, top, mode, correction, route_scale, groups, keep, vec, bias, side);
     }));
   }
   if (fms_launch_status("route")) return 1;
@@ -733,13 +755,14 @@ FMS_API int fms_gated_clamped(const void* gu, void* out, int dtype, int n_rows, 
   return fms_launch_status("gated_clamped");
 }
 
-// weight: [n_tokens, top] float32 that multiply the pairs' rows, or null for their plain sum
+// weight: [n_tokens, top] float32 that multiply the pairs' rows, or null for their plain sum.  shared: [n_tokens, dim] that
+// every token adds, times side [n_tokens] float32 where that is given (null: nothing / as it is)
 FMS_API int fms_route_gather(const void* ys, int dtype, const int* row_of_pair, void* out, int n_tokens, int dim, int top,
-                             const float* weight, cudaStream_t stream) {
+                             const float* weight, const void* shared, const float* side, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   FMS_DISPATCH_DTYPE(dtype, T,
                      fms_launch(route_gather_kernel<T>, dim3(n_tokens), dim3(256), 2 * sizeof(int) * top, stream, (const T*)ys, row_of_pair,
-                                (T*)out, dim, top, n_tokens * top, weight,
-                                dim % 8 == 0 && ((uintptr_t)ys & 15) == 0 && ((uintptr_t)out & 15) == 0 ? 1 : 0));
+                                (T*)out, dim, top, n_tokens * top, weight, (const T*)shared, side,
+                                dim % 8 == 0 && (((uintptr_t)ys | (uintptr_t)out | (uintptr_t)shared) & 15) == 0 ? 1 : 0));
   return fms_launch_status("route_gather");
 }

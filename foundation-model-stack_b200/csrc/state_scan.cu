@@ -15,7 +15,9 @@
 //                       a and b from exponential gates under a running maximum m (m' = max(f + m, i), a = exp(f + m - m'),
 //                       b = exp(i - m')), a normalizer n = a n + b k and o = S^T q / (max(|n.q|, exp(-m')) + 1e-6);
 //                       linear_prepare makes q, k, v float32 (an activation, a factor on q), exp_gates walks the maxima
-//                       and leaves (a, b, exp(-m')) for every token; the scan carries n beside its state columns
+//                       and leaves (a, b, exp(-m')) for every token; the scan carries n beside its state columns;
+//                       or with one decay a key channel, S = diag(a) S + k v^T, a = sigmoid(W u + bias)^(1 / tau), all of
+//                       which gla_prepare makes ready for every token before the scan starts
 //   gated_group_rmsnorm rows cut into groups, each divided by its own root mean square, times a weight; a gate
 //                       multiplies either before the norm (silu) or after it (sigmoid)
 //
@@ -596,19 +598,100 @@ __global__ void exp_gates_kernel(const T* gate_raw, int stride, const float* bia
   if (write_state && lane == 0) st[dim] = m;
 }
 
+// What a scan under one decay a key channel reads, made ready for every token at once: q | k | v in float32 (q times
+// q_scale) and the decays sigmoid(w . u + bias)^(1 / tau), u being `rank` columns of the projection's rows.  A block takes
+// GLA_TOKENS tokens and either 128 channels of the decays (the first `decay_blocks` of its grid column: a thread holds its
+// channel's row of w against all of them) or a run of 512 columns of q | k | v.  The logarithm of a decay is taken in
+// double and the decay rounded once: its error compounds over a sequence.
+constexpr int GLA_TOKENS = 8, GLA_THREADS = 128;
+
+template <typename TW> __device__ __forceinline__ void load_row8(const TW* p, float (&v)[8]) {
+  float a[4], b[4];
+  load_channels<4>(p, a);
+  load_channels<4>(p + 4, b);
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    v[k] = a[k];
+    v[4 + k] = b[k];
+  }
+}
+
+template <typename T, typename TW>
+__global__ void __launch_bounds__(GLA_THREADS) gla_prepare_kernel(const T* proj, int stride, int u_col, int rank, const TW* w,
+                                                                  const float* bias, double inv_tau, float* decay,
+                                                                  int channels, int decay_blocks, float* qkv, int cols,
+                                                                  int q_cols, float q_scale, int n_tokens, int vec_w, int vec) {
+  extern __shared__ __align__(16) float us[];  // [GLA_TOKENS][rank]
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t0 = blockIdx.x * GLA_TOKENS, tn = min(GLA_TOKENS, n_tokens - t0);
+  if ((int)blockIdx.y < decay_blocks) {
+    for (int i = threadIdx.x; i < GLA_TOKENS * rank; i += blockDim.x) {
+      const int t = i / rank, r = i - t * rank;
+      us[i] = t < tn ? to_f32(proj[(size_t)(t0 + t) * stride + u_col + r]) : 0.f;
+    }
+    __syncthreads();
+    const int c = blockIdx.y * GLA_THREADS + threadIdx.x;
+    if (c >= channels) return;
+    const TW* row = w + (size_t)c * rank;
+    float z[GLA_TOKENS];
+#pragma unroll
+    for (int t = 0; t < GLA_TOKENS; ++t) z[t] = 0.f;
+    if (vec_w) {
+      for (int r = 0; r < rank; r += 8) {
+        float wv[8];
+        load_row8(row + r, wv);
+#pragma unroll
+        for (int t = 0; t < GLA_TOKENS; ++t)
+#pragma unroll
+          for (int k = 0; k < 8; ++k) z[t] = fmaf(wv[k], us[t * rank + r + k], z[t]);
+      }
+    } else {
+      for (int r = 0; r < rank; ++r) {
+        const float wr = to_f32(row[r]);
+#pragma unroll
+        for (int t = 0; t < GLA_TOKENS; ++t) z[t] = fmaf(wr, us[t * rank + r], z[t]);
+      }
+    }
+    const float b = bias[c];
+#pragma unroll
+    for (int t = 0; t < GLA_TOKENS; ++t)
+      if (t < tn) decay[(size_t)(t0 + t) * channels + c] = (float)exp(-softplus_d(-(double)(z[t] + b)) * inv_tau);
+    return;
+  }
+  const int c = (((int)blockIdx.y - decay_blocks) * GLA_THREADS + threadIdx.x) * 4;
+  if (c >= cols) return;
+  for (int t = 0; t < tn; ++t) {
+    const T* src = proj + (size_t)(t0 + t) * stride + c;
+    float* dst = qkv + (size_t)(t0 + t) * cols + c;
+    if (vec) {  // cols a multiple of 4
+      float v[4];
+      load_channels<4>(src, v);
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+        if (c + k < q_cols) v[k] *= q_scale;
+      *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+    } else {
+      for (int k = 0; k < 4 && c + k < cols; ++k) dst[k] = to_f32(src[k]) * (c + k < q_cols ? q_scale : 1.f);
+    }
+  }
+}
+
 // qkv [tokens, 2 heads * dim + heads * vdim] float32: q | k | v, head by head; o [tokens, heads * vdim].
-// GATED: per token and head (a, b, e) in gates [tokens, heads, 3]: S = a S + b k v^T, n = a n + b k,
+// KIND 1 (gated): per token and head (a, b, e) in gates [tokens, heads, 3]: S = a S + b k v^T, n = a n + b k,
 // o = S^T q / (max(|n.q|, e) + 1e-6).  Every thread walks its rows of n beside its rows of the state columns (n is
 // the state column of a value that is always one), so that a column group has n.q from the same shuffles as its sums
 // and no thread waits for another group; n before the step comes from norm_in [sequences, heads, dim], and the first
 // column group of a head's first block leaves the new n in norm_state [slots, heads, dim + 1].
-// Else one decay a head (decay [heads]): S = decay S + k v^T, o = S^T q.
-template <int NP, int VP, int PARTS, bool GATED>
+// KIND 2: one decay a token and key channel (gates [tokens, heads * dim]): S = diag(a) S + k v^T, o = S^T q.
+// KIND 0: one decay a head (decay [heads]): S = decay S + k v^T, o = S^T q.
+template <int NP, int VP, int PARTS, int KIND>
 __global__ void __launch_bounds__(SCAN_THREADS) decay_scan_kernel(const float* qkv, const float* gates, const float* decay,
                                                                   float* state, const float* norm_in, float* norm_state,
                                                                   float* o, const int* first_row, const int* slots,
                                                                   int heads, int dim, int vdim, int write_state,
-                                                                  int n_slots, int vec_qk, int vec_v) {
+                                                                  int n_slots, int vec_qk, int vec_v, int vec_g) {
+  constexpr bool GATED = KIND == 1, CHANNEL = KIND == 2;
   constexpr int GROUPS = SCAN_THREADS / PARTS, NPAD = RowLayout<NP, PARTS>::ROW, RUN = RowLayout<NP, PARTS>::RUN, VB = GROUPS * VP;
   extern __shared__ __align__(16) float smem[];
   pdl_launch_dependents();
@@ -619,7 +702,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) decay_scan_kernel(const float* q
   if (!FMS_IN(slot, n_slots)) return;
   const int lo = first_row[seq], hi = first_row[seq + 1];
   const int row_w = 2 * heads * dim + heads * vdim;
-  constexpr int STAGE = CH * (2 * NPAD + VB + 4);
+  constexpr int STAGE = CH * ((CHANNEL ? 3 : 2) * NPAD + VB + 4);
   const int cols = min(VB, vdim - v0);
   if (dim != PARTS * NP || cols != VB)
     for (int i = tid; i < 2 * STAGE; i += blockDim.x) smem[i] = 0.f;  // the padding stays zero from here on
@@ -631,7 +714,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) decay_scan_kernel(const float* q
   }
   float nn[GATED ? NP : 1];
   if constexpr (GATED) load_state<NP, PARTS>(norm_in + ((size_t)seq * heads + head) * dim, part, dim, true, nn);
-  const float fixed = GATED ? 1.f : decay[head];
+  const float fixed = KIND != 0 ? 1.f : decay[head];
   __syncthreads();
   auto issue = [&](int c0, int stage) {
     const int cn = min(CH, hi - c0);
@@ -641,6 +724,8 @@ __global__ void __launch_bounds__(SCAN_THREADS) decay_scan_kernel(const float* q
     stage_runs<NP, PARTS>(base + CH * NPAD, src + (size_t)(heads + head) * dim, row_w, cn, dim, vec_qk);
     stage_rows(base + 2 * CH * NPAD, VB, src + 2 * (size_t)heads * dim + (size_t)head * vdim + v0, row_w, cn, cols, vec_v);
     if (GATED) stage_rows(base + 2 * CH * NPAD + CH * VB, 4, gates + ((size_t)c0 * heads + head) * 3, (size_t)heads * 3, cn, 3, false);
+    if (CHANNEL)
+      stage_runs<NP, PARTS>(base + CH * (2 * NPAD + VB + 4), gates + ((size_t)c0 * heads + head) * dim, (size_t)heads * dim, cn, dim, vec_g);
     cp_async_commit();
   };
   if (lo < hi) issue(lo, 0);
@@ -655,6 +740,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) decay_scan_kernel(const float* q
     const float* sk = sq + CH * NPAD;
     const float* sv = sk + CH * NPAD;
     const float* sg = sv + CH * VB;
+    const float* sa = sg + CH * 4;
     // two tokens an iteration and two partial sums a column (even and odd rows): a token's loads and sums do not
     // wait for the token before it, only its state values do
 #pragma unroll 2
@@ -663,6 +749,8 @@ __global__ void __launch_bounds__(SCAN_THREADS) decay_scan_kernel(const float* q
       load_run<NP>(sk + t * NPAD + part * RUN, k);
       load_run<NP>(sq + t * NPAD + part * RUN, q);
       const float a = GATED ? sg[t * 4] : fixed;
+      float ch[CHANNEL ? NP : 1];
+      if constexpr (CHANNEL) load_run<NP>(sa + t * NPAD + part * RUN, ch);
       const float b = GATED ? sg[t * 4 + 1] : 1.f;
       float acc[VP], odd[VP], val[VP], nq = 0.f, nq_odd = 0.f;
 #pragma unroll
@@ -673,10 +761,11 @@ __global__ void __launch_bounds__(SCAN_THREADS) decay_scan_kernel(const float* q
 #pragma unroll
       for (int j = 0; j < NP; j += 2) {
         const float k0 = k[j], q0 = q[j], k1 = k[j + 1], q1 = q[j + 1];
+        const float a0 = CHANNEL ? ch[CHANNEL ? j : 0] : a, a1 = CHANNEL ? ch[CHANNEL ? j + 1 : 0] : a;
 #pragma unroll
         for (int i = 0; i < VP; ++i) {
-          s[i][j] = fmaf(a, s[i][j], k0 * val[i]);
-          s[i][j + 1] = fmaf(a, s[i][j + 1], k1 * val[i]);
+          s[i][j] = fmaf(a0, s[i][j], k0 * val[i]);
+          s[i][j + 1] = fmaf(a1, s[i][j + 1], k1 * val[i]);
           acc[i] = fmaf(s[i][j], q0, acc[i]);
           odd[i] = fmaf(s[i][j + 1], q1, odd[i]);
         }
@@ -972,10 +1061,30 @@ FMS_API int fms_linear_prepare(const void* proj, int dtype, int stride, float* o
   return fms_launch_status("linear_prepare");
 }
 
+// What fms_decay_scan reads under one decay a key channel: q | k | v of a step's rows in float32 (the first q_cols columns
+// times q_scale) and decays [tokens, channels] = sigmoid(w u + bias)^(1 / tau), u = columns u_col .. u_col + rank of the
+// rows, w [channels, rank], bias [channels] float32
+FMS_API int fms_gla_prepare(const void* proj, int dtype, int stride, int u_col, int rank, const void* w, int w_dtype,
+                            const float* bias, float tau, float* decay, int channels, float* qkv, int n_tokens, int cols,
+                            int q_cols, float q_scale, cudaStream_t stream) {
+  if (n_tokens <= 0 || cols <= 0) return 0;
+  if (rank <= 0 || rank > 1024 || channels <= 0 || !(tau > 0.f)) return fms_fail("gla_prepare: rank %d (up to 1024), %d channels, tau %f", rank, channels, tau);
+  const size_t item = dtype == FMS_BF16 ? 2 : 4, w_item = w_dtype == FMS_BF16 ? 2 : 4;
+  const int vec = cols % 4 == 0 && stride % 4 == 0 && (uintptr_t)proj % (4 * item) == 0 && (uintptr_t)qkv % 16 == 0;
+  const int vec_w = rank % 8 == 0 && (uintptr_t)w % (4 * w_item) == 0;
+  const int decay_blocks = (channels + GLA_THREADS - 1) / GLA_THREADS;
+  const dim3 grid((n_tokens + GLA_TOKENS - 1) / GLA_TOKENS, decay_blocks + (cols + 4 * GLA_THREADS - 1) / (4 * GLA_THREADS));
+  FMS_DISPATCH_DTYPE(dtype, T, FMS_DISPATCH_DTYPE(w_dtype, TW,
+                     fms_launch(gla_prepare_kernel<T, TW>, grid, dim3(GLA_THREADS), (size_t)GLA_TOKENS * rank * sizeof(float), stream,
+                                (const T*)proj, stride, u_col, rank, (const TW*)w, bias, 1.0 / (double)tau, decay, channels,
+                                decay_blocks, qkv, cols, q_cols, q_scale, n_tokens, vec_w, vec)));
+  return fms_launch_status("gla_prepare");
+}
+
 // qkv [tokens, 2 heads * dim + heads * vdim] float32.  With gate_raw (columns [i: heads | f: heads] of rows of
 // gate_stride values, bias [2 heads], cap): exponential gates, with normalizer and running maximum in norm_state
 // [slots, heads, dim + 1]; gates [tokens, heads, 3] and norm_in [sequences, heads, dim] are float32 scratch of the
-// caller's.  Without: decay [heads].
+// caller's.  With gates but no gate_raw: one decay a token and key channel, gates [tokens, heads * dim].  Else: decay [heads].
 FMS_API int fms_decay_scan(const float* qkv, const void* gate_raw, int dtype, int gate_stride, const float* gate_bias,
                            float cap, float* gates, float* norm_in, const float* decay, float* state, float* norm_state, float* o,
                            const int* first_row, const int* slots, int n_tokens, int n_seqs, int heads, int dim, int vdim,
@@ -985,7 +1094,8 @@ FMS_API int fms_decay_scan(const float* qkv, const void* gate_raw, int dtype, in
     return fms_fail("decay_scan: %d heads, dim %d (up to 256), vdim %d", heads, dim, vdim);
   const bool gated = gate_raw != nullptr;
   if (gated && (!gate_bias || !gates || !norm_in || !norm_state || !(cap > 0.f))) return fms_fail("decay_scan: gates without bias, scratch, normalizer or cap");
-  if (!gated && !decay) return fms_fail("decay_scan: neither gates nor decays");
+  const bool channel = !gated && gates != nullptr;
+  if (!gated && !channel && !decay) return fms_fail("decay_scan: neither gates nor decays");
   const long row_w = 2L * heads * dim + (long)heads * vdim;
   if (gated) {
     FMS_DISPATCH_DTYPE(dtype, T, fms_launch(exp_gates_kernel<T>, dim3((n_seqs * heads + 3) / 4), dim3(128), 0, stream,
@@ -999,18 +1109,22 @@ FMS_API int fms_decay_scan(const float* qkv, const void* gate_raw, int dtype, in
   const int vb = SCAN_THREADS / shape.parts * shape.vp;  // value columns of a block
   const int vec_qk = rows_allow_16(qkv, 0, row_w, dim) && shape.np % 4 == 0;
   const int vec_v = rows_allow_16(qkv, 2L * heads * dim, row_w, vdim) && vdim % vb == 0 && vb % 4 == 0;
+  const int vec_g = channel && rows_allow_16(gates, 0, (long)heads * dim, dim) && shape.np % 4 == 0;
   const dim3 grid(n_seqs, heads, (vdim + vb - 1) / vb), block(SCAN_THREADS);
-#define FMS_LAUNCH_G(NP, VP, PARTS, GATED)                                                                              \
+#define FMS_LAUNCH_G(NP, VP, PARTS, KIND)                                                                               \
   do {                                                                                                                  \
-    const size_t smem = ((size_t)2 * CH * (2 * RowLayout<NP, PARTS>::ROW + SCAN_THREADS / PARTS * VP + 4)) * sizeof(float); \
-    cudaFuncSetAttribute(decay_scan_kernel<NP, VP, PARTS, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-    fms_launch(decay_scan_kernel<NP, VP, PARTS, GATED>, grid, block, smem, stream, qkv, (const float*)gates, decay, state, \
-               (const float*)norm_in, norm_state, o, first_row, slots, heads, dim, vdim, write_state, n_slots, vec_qk, vec_v); \
+    const size_t smem = ((size_t)2 * CH * ((KIND == 2 ? 3 : 2) * RowLayout<NP, PARTS>::ROW + SCAN_THREADS / PARTS * VP + 4)) * sizeof(float); \
+    cudaFuncSetAttribute(decay_scan_kernel<NP, VP, PARTS, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    fms_launch(decay_scan_kernel<NP, VP, PARTS, KIND>, grid, block, smem, stream, qkv, (const float*)gates, decay, state, \
+               (const float*)norm_in, norm_state, o, first_row, slots, heads, dim, vdim, write_state, n_slots, vec_qk, vec_v, vec_g); \
   } while (0)
-#define FMS_LAUNCH_T(NP, VP, PARTS) FMS_LAUNCH_G(NP, VP, PARTS, true)
-#define FMS_LAUNCH_F(NP, VP, PARTS) FMS_LAUNCH_G(NP, VP, PARTS, false)
+#define FMS_LAUNCH_F(NP, VP, PARTS) FMS_LAUNCH_G(NP, VP, PARTS, 0)
+#define FMS_LAUNCH_T(NP, VP, PARTS) FMS_LAUNCH_G(NP, VP, PARTS, 1)
+#define FMS_LAUNCH_C(NP, VP, PARTS) FMS_LAUNCH_G(NP, VP, PARTS, 2)
   if (gated) FMS_SCAN_SHAPES(FMS_LAUNCH_T);
+  else if (channel) FMS_SCAN_SHAPES(FMS_LAUNCH_C);
   else FMS_SCAN_SHAPES(FMS_LAUNCH_F);
+#undef FMS_LAUNCH_C
 #undef FMS_LAUNCH_T
 #undef FMS_LAUNCH_F
 #undef FMS_LAUNCH_G

@@ -14,6 +14,7 @@ from ..parts.base import Part
 from ..parts import block as _blocks  # noqa: F401  (registers the built-in arrangement)
 from ..parts import embedding as _embeddings  # noqa: F401  (registers the built-in embeddings)
 from ..parts.registry import build_block, build_embedding, build_norm
+from ..parts.streams import StreamSet
 
 
 def _add_path(root: Part, path: str, part: Part) -> Part:
@@ -71,11 +72,15 @@ class Decoder(Part):
         if getattr(batch, "scratch", None) is not None:
             batch.scratch.clear()  # nothing of an earlier step with the same arrays (a decode step) is kept
         residual = self.embedding.forward(batch, cache.layer_view("embedding"), self.spec.embedding_scale)
+        if self.spec.streams:
+            residual = StreamSet(residual, self.spec.streams)
         pending = None
         for call in self.spec.schedule:
             view = cache.layer_view(call.cache_layer)
             pending = self.blocks[call.layer].forward(residual, pending, batch, view, call.writes_cache, self.dtype)
         h = self.final_norm.apply(residual, pending, self.dtype, rows=batch.want_rows)
+        if self.spec.logit_softcap > 0.0:
+            return ops.capped_logits(h, self.head_weight(), self.spec.logit_scale, self.spec.logit_softcap)
         logits = ops.linear(h, self.head_weight(), None, torch.float32)
         if self.spec.logit_scale != 1.0:
             logits.mul_(self.spec.logit_scale)

@@ -46,6 +46,8 @@ _SIGNATURES = {
     "fms_linear_bf16_skinny": [_P, _P, _P, _P, _I, _I, _I, _I, _P],
     "fms_token_gate_bf16_skinny": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
     "fms_grouped_bf16_skinny": [_P, _P, _P, _P, _I, _I, _I, _I, _P],
+    "fms_linear_act_bf16_skinny": [_P, _P, _P, _P, _I, _I, _I, _I, _P],
+    "fms_linear_cap_bf16_skinny": [_P, _P, _P, _I, _I, _I, _F, _F, _P],
     "fms_glu_bf16_skinny": [_P, _P, _P, _P, _I, _I, _I, _I, _P],
     "fms_qkv_rope_store_bf16_skinny": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P,
                                        _I, _I, _I, _P],
@@ -54,6 +56,7 @@ _SIGNATURES = {
     "fms_qkv_rope_store_bf16_mid": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P,
                                     _I, _I, _I, _P],
     "fms_gemm_bf16_tc": [_P, _P, _P, _P, _I, _I, _I, _I, _P, _P],
+    "fms_linear_act_bf16_tc": [_P, _P, _P, _P, _I, _I, _I, _I, _P, _P],
     "fms_glu_bf16_tc": [_P, _P, _P, _P, _I, _I, _I, _I, _P, _P],
     "fms_qkv_rope_store_bf16_tc": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P,
                                    _I, _I, _I, _P],
@@ -61,8 +64,8 @@ _SIGNATURES = {
     "fms_normed_add_rmsnorm": [_P, _P, _I, _P, _F, _F, _P, _F, _F, _I, _P, _I, _P, _I, _I, _I, _P],
     "fms_mingru_scan": [_P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _P, _P, _I, _P, _P],
     "fms_grouped_linear": [_P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _L, _L, _L, _L, _I, _F, _F, _I, _P],
-    "fms_route": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _F, _I, _I, _P, _P],
-    "fms_route_gather": [_P, _I, _P, _P, _I, _I, _I, _P, _P],
+    "fms_route": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _F, _I, _I, _P, _P, _P, _P],
+    "fms_route_gather": [_P, _I, _P, _P, _I, _I, _I, _P, _P, _P, _P],
     "fms_relu_squared": [_P, _I, _L, _P],
     "fms_gated_clamped": [_P, _P, _I, _I, _I, _F, _F, _P],
     "fms_latent_attention_prefill_bf16": [_P, _P, _P, _P, _L, _P, _I, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I,
@@ -79,6 +82,10 @@ _SIGNATURES = {
                              _I, _I, _I, _I, _I, _P, _I, _I, _I, _P, _I, _F, _P],
     "fms_sigmoid_gate": [_P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _I, _P],
     "fms_normed_add_norm": [_P, _P, _F, _P, _F, _P, _F, _P, _F, _I, _P, _F, _I, _P, _P, _F, _P, _I, _P, _I, _I, _I, _P],
+    "fms_stream_mix_norm": [_P, _I, _P, _P, _P, _P, _P, _F, _P, _I, _P, _I, _I, _I, _I, _P],
+    "fms_activation": [_P, _I, _I, _L, _P],
+    "fms_scale_cap": [_P, _F, _F, _L, _P],
+    "fms_gla_prepare": [_P, _I, _I, _I, _I, _P, _I, _P, _F, _P, _I, _P, _I, _I, _I, _F, _P],
     "fms_linear_prepare": [_P, _I, _I, _P, _I, _I, _I, _F, _I, _P],
     "fms_decay_scan": [_P, _P, _I, _I, _P, _F, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "fms_attention_prefill_sink": [_P, _P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P,
@@ -368,6 +375,34 @@ def parts_group_rmsnorm(residual: torch.Tensor, parts, gains, eps: float, groups
     return outs
 
 
+def stream_mix_norm(streams, delta: Optional[torch.Tensor], on: Optional[torch.Tensor], w_in: torch.Tensor,
+                    gain: Optional[torch.Tensor], eps: float, out_dtype: torch.dtype,
+                    rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Several residual streams X_s a token (a ``parts.streams.StreamSet``, float32).  First X_t becomes
+    sum_s mix[s, t] X_s + w_out[t] * delta, in place, where there is a ``delta`` [tokens, dim] in the compute dtype
+    (``on`` float32: mix [streams, streams], from and to, then w_out [streams]); then returns u / sqrt(mean(u^2) + eps) *
+    gain for u = sum_s w_in[s] X_s in ``out_dtype`` (``gain`` float32 [dim]; None: u).  With ``rows`` only those tokens are
+    computed and the streams are not written."""
+    start, n_streams = streams.start, streams.streams
+    n_all, dim = start.shape
+    n = rows.shape[0] if rows is not None else n_all
+    if start.dtype != torch.float32 or (delta is not None and (delta.dtype != out_dtype or tuple(delta.shape) != (n_all, dim))):
+        raise KernelError(f"stream_mix_norm: the streams are float32, a sublayer's output {out_dtype} [{n_all}, {dim}]")
+    if w_in.dtype != torch.float32 or w_in.shape[0] != n_streams or (gain is not None and (gain.dtype != torch.float32 or gain.shape[0] != dim)) \
+            or (delta is not None and (on is None or on.dtype != torch.float32 or on.numel() != n_streams * (n_streams + 1))):
+        raise KernelError(f"stream_mix_norm: float32 weights of {n_streams} streams and a gain of {dim}")
+    src, src_streams = (start, 1) if streams.rows is None else (streams.rows, n_streams)
+    dst = None
+    if delta is not None and rows is None:
+        if streams.rows is None:
+            streams.rows = torch.empty((n_all, n_streams, dim), dtype=torch.float32, device=start.device)
+        dst = streams.rows
+    out = torch.empty((n, dim), dtype=out_dtype, device=start.device)
+    _call("elementwise", "fms_stream_mix_norm", _ptr(src), src_streams, _ptr(dst), _ptr(delta), _ptr(on), _ptr(w_in), _ptr(gain),
+          float(eps), _ptr(out), _code(out_dtype), _ptr(rows), n, dim, n_streams, n_all, _stream())
+    return out
+
+
 def cast_rows(x: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
     """Float32 rows in ``dtype`` (the same tensor where that is float32)."""
     if dtype == torch.float32:
@@ -411,6 +446,19 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] =
         return y if bias is None else y + bias.float()
     b = None if bias is None else bias.to(torch.bfloat16)
     return torch.nn.functional.linear(x, weight, b)
+
+
+def capped_logits(x: torch.Tensor, weight: torch.Tensor, scale: float, cap: float) -> torch.Tensor:
+    """Float32 logits cap * tanh(scale * x weight^T / cap) (``cap`` 0: without the cap): for a few bfloat16 rows in the
+    product's epilogue, else a pass over the product's results."""
+    if x.dtype == weight.dtype == torch.bfloat16 and x.shape[0] <= SKINNY_ROWS and weight.shape[1] % 8 == 0:
+        y = torch.empty((x.shape[0], weight.shape[0]), dtype=torch.float32, device=x.device)
+        _call("gemm_bf16_skinny", "fms_linear_cap_bf16_skinny", _ptr(x), _ptr(weight), _ptr(y), x.shape[0], weight.shape[0],
+              weight.shape[1], float(scale), float(cap), _stream())
+        return y
+    y = linear(x, weight, None, torch.float32)
+    _call("elementwise", "fms_scale_cap", _ptr(y), float(scale), float(cap), y.numel(), _stream())
+    return y
 
 
 # Rows from which the tcgen05 kernel with the tokens on the instruction's rows (gemm_bf16_tc.cu) is used instead of the
@@ -506,6 +554,28 @@ def gated_linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Ten
             and (x.shape[0] + 255) // 256 * 256 <= TENSOR_CORE_MAX_PADDING * x.shape[0]):
         return gated_linear_tensor_core(x, weight, bias, activation)
     return gated_activation(linear(x, weight, bias), activation)
+
+
+def activated_linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], activation: int) -> torch.Tensor:
+    """act(x weight^T + bias): the first product of an ungated feed-forward.  A few bfloat16 rows: the weight-streaming kernel
+    with the activation in its epilogue; many, where its tiles fit (as for the gated product): the tcgen05 kernel with
+    the activation in its epilogue; else the product and then the activation in place."""
+    own = x.dtype == weight.dtype == torch.bfloat16 and weight.shape[1] % 8 == 0 and (bias is None or bias.dtype == torch.bfloat16) \
+        and activation <= 3
+    if own and x.shape[0] <= SKINNY_ROWS:
+        y = torch.empty((x.shape[0], weight.shape[0]), dtype=x.dtype, device=x.device)
+        _call("gemm_bf16_skinny", "fms_linear_act_bf16_skinny", _ptr(x), _ptr(weight), _ptr(bias), _ptr(y), x.shape[0],
+              weight.shape[0], weight.shape[1], int(activation), _stream())
+        return y
+    if (own and _tensor_core_fits(x, weight, bias, TENSOR_CORE_ROWS_GLU)
+            and (x.shape[0] + 255) // 256 * 256 <= TENSOR_CORE_MAX_PADDING * x.shape[0]):
+        y = torch.empty((x.shape[0], weight.shape[0]), dtype=x.dtype, device=x.device)
+        _call("gemm_bf16_tc", "fms_linear_act_bf16_tc", _ptr(x), _ptr(weight), _ptr(bias), _ptr(y), x.shape[0], weight.shape[0],
+              weight.shape[1], int(activation), _ptr(error_flag(x.device)), _stream())
+        return y
+    y = linear(x, weight, bias)
+    _call("elementwise", "fms_activation", _ptr(y), _code(y.dtype), int(activation), y.numel(), _stream())
+    return y
 
 
 def gated_activation(gate_up: torch.Tensor, activation: int) -> torch.Tensor:
@@ -885,6 +955,33 @@ def delta_rule_scan(qkv: torch.Tensor, proj: torch.Tensor, beta_offset: int, a_r
     return o
 
 
+def gla_scan(proj: torch.Tensor, state: torch.Tensor, batch, heads: int, dim: int, vdim: int, rank_offset: int,
+             decay_weight: torch.Tensor, decay_bias: torch.Tensor, tau: float, q_scale: float,
+             writes_state: bool = True) -> torch.Tensor:
+    """A state matrix per head with one decay a token and key channel, over each sequence's rows: S = diag(a) S + k v^T;
+    o = S^T (q_scale q), a = sigmoid(decay_weight u + decay_bias)^(1 / tau).  The columns of ``proj`` are [q: heads x dim |
+    k: heads x dim | v: heads x vdim | ...], u its columns ``rank_offset .. rank_offset + rank``; ``decay_weight``
+    [heads * dim, rank], ``decay_bias`` float32 [heads * dim]; ``state`` float32 [slots, heads, vdim, dim].  Returns o float32
+    [tokens, heads * vdim]."""
+    n = proj.shape[0]
+    cols, channels = heads * (2 * dim + vdim), heads * dim
+    rank = decay_weight.shape[1]
+    if state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, vdim, dim) or proj.shape[1] < max(cols, rank_offset + rank):
+        raise KernelError("gla_scan: proj [tokens, q | k | v | ... | u ...], state float32 [slots, heads, vdim, dim]")
+    if decay_weight.shape[0] != channels or decay_bias.dtype != torch.float32 or decay_bias.shape[0] != channels:
+        raise KernelError("gla_scan: a row of the decays' matrix and a float32 bias for every head and key channel")
+    qkv = torch.empty((n, cols), dtype=torch.float32, device=proj.device)
+    decay = torch.empty((n, channels), dtype=torch.float32, device=proj.device)
+    _call("state_scan", "fms_gla_prepare", _ptr(proj), _code(proj.dtype), proj.shape[1], int(rank_offset), rank, _ptr(decay_weight),
+          _code(decay_weight.dtype), _ptr(decay_bias), float(tau), _ptr(decay), channels, _ptr(qkv), n, cols, channels,
+          float(q_scale), _stream())
+    o = torch.empty((n, heads * vdim), dtype=torch.float32, device=proj.device)
+    _call("state_scan", "fms_decay_scan", _ptr(qkv), None, _code(proj.dtype), 0, None, 0.0, _ptr(decay), None, None, _ptr(state),
+          None, _ptr(o), _ptr(batch.first_row), _ptr(batch.slots), n, batch.n_seqs, heads, dim, vdim,
+          1 if writes_state else 0, state.shape[0], _stream())
+    return o
+
+
 ACT_NONE, ACT_SILU = 0, 1
 
 
@@ -987,14 +1084,15 @@ class Routing:
     matrix, and the sorted, weighted rows themselves."""
 
     __slots__ = ("expert", "weight", "offsets", "tile_first", "row_of_pair", "group_of_row", "rows", "top", "experts",
-                 "weights_on_output")
+                 "weights_on_output", "side")
 
 
-ROUTE_SIGMOID, ROUTE_SOFTMAX, ROUTE_SIGMOID_GROUPS = 0, 1, 2
+ROUTE_SIGMOID, ROUTE_SOFTMAX, ROUTE_SIGMOID_GROUPS, ROUTE_SOFTMAX_CHOSEN = 0, 1, 2, 3
 
 
 def route(x: torch.Tensor, router: torch.Tensor, top: int, mode: int = ROUTE_SIGMOID,
-          correction: Optional[torch.Tensor] = None, route_scale: float = 1.0, groups: int = 1, keep: int = 1) -> Routing:
+          correction: Optional[torch.Tensor] = None, route_scale: float = 1.0, groups: int = 1, keep: int = 1,
+          bias: Optional[torch.Tensor] = None, side: bool = False) -> Routing:
     """``ROUTE_SIGMOID``: scores sigmoid(x router^T) in float32; every token's ``top`` best experts; rows
     weight * x[token] sorted by expert.  ``ROUTE_SOFTMAX``: scores softmax(x router^T) over all experts; the ``top``
     experts with the largest score + ``correction`` [experts] (float32, or None) are the token's; its weights are their
@@ -1002,11 +1100,17 @@ def route(x: torch.Tensor, router: torch.Tensor, top: int, mode: int = ROUTE_SIG
     ``route_gather`` multiplies the experts' results by the weights.  ``ROUTE_SIGMOID_GROUPS``: scores sigmoid(x
     router^T); the choice is by score + ``correction`` among the experts of the ``keep`` best of ``groups`` equal groups of
     neighbours (a group's score: the sum of its two largest choice scores); the weights are the chosen scores (without
-    the correction) times ``route_scale``, and multiply the results as with ``ROUTE_SOFTMAX``."""
-    if correction is not None and (correction.dtype != torch.float32 or correction.shape[0] != router.shape[0]):
+    the correction) times ``route_scale``, and multiply the results as with ``ROUTE_SOFTMAX``.  ``ROUTE_SOFTMAX_CHOSEN``: the
+    ``top`` largest logits are chosen, the weights are the softmax over those alone times ``route_scale``, and multiply the
+    results.  ``bias`` [experts] float32 is added to the logits first.  ``side``: the router's matrix has a row behind the
+    experts' and ``Routing.side`` [tokens] float32 = sigmoid(x . that row), which ``route_gather`` takes for a unit that
+    every token uses."""
+    if bias is not None and (bias.dtype != torch.float32 or bias.shape[0] != router.shape[0] - (1 if side else 0)):
+        raise KernelError("route: the bias is float32, one number an expert")
+    if correction is not None and (correction.dtype != torch.float32 or correction.shape[0] != router.shape[0] - (1 if side else 0)):
         raise KernelError("route: the correction is float32, one number an expert")
     n, dim = x.shape
-    experts = router.shape[0]
+    experts = router.shape[0] - (1 if side else 0)
     dev = x.device
     r = Routing()
     r.top, r.experts = top, experts
@@ -1020,6 +1124,7 @@ def route(x: torch.Tensor, router: torch.Tensor, top: int, mode: int = ROUTE_SIG
     r.offsets = ints[o + experts + 1: o + 2 * (experts + 1)]
     r.tile_first = ints[o + 2 * (experts + 1): o + 3 * (experts + 1)]
     r.weight = torch.empty((n, top), dtype=torch.float32, device=dev)
+    r.side = torch.empty((n,), dtype=torch.float32, device=dev) if side else None
     r.rows = torch.empty((n * top, dim), dtype=x.dtype, device=dev)
     # many bfloat16 rows: the logits from the library's product with float32 results (bfloat16 factors are exact in it)
     logits = None
@@ -1029,7 +1134,7 @@ def route(x: torch.Tensor, router: torch.Tensor, top: int, mode: int = ROUTE_SIG
     _call("grouped", "fms_route", _ptr(x), _code(x.dtype), _ptr(router), _code(router.dtype), _ptr(r.expert),
           _ptr(r.weight), _ptr(counts), _ptr(r.offsets), _ptr(r.tile_first), _ptr(r.row_of_pair), _ptr(r.group_of_row),
           _ptr(r.rows), n, dim, experts, top, int(mode), _ptr(correction), float(route_scale), int(groups), int(keep),
-          _ptr(logits), _stream())
+          _ptr(logits), _ptr(bias), _ptr(r.side), _stream())
     global launches
     launches += 2
     return r
@@ -1072,13 +1177,17 @@ def routed_linear(rows: torch.Tensor, weight: torch.Tensor, routing: Routing, gl
     return y
 
 
-def route_gather(ys: torch.Tensor, routing: Routing) -> torch.Tensor:
+def route_gather(ys: torch.Tensor, routing: Routing, every: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[token] = the sum of its pairs' rows of ``ys`` (each times its weight where the routing left the weights for
-    the experts' results), float32, in the order of its choices."""
+    the experts' results), float32, in the order of its choices; plus the token's row of ``every`` [tokens, dim], times
+    ``routing.side`` where the routing has it."""
+    if every is not None and (every.dtype != ys.dtype or tuple(every.shape) != (ys.shape[0] // routing.top, ys.shape[1])):
+        raise KernelError(f"route_gather: rows {ys.dtype} {tuple(ys.shape)} of {routing.top} a token, beside {every.dtype} {tuple(every.shape)}")
     n = ys.shape[0] // routing.top
     out = torch.empty((n, ys.shape[1]), dtype=ys.dtype, device=ys.device)
     _call("grouped", "fms_route_gather", _ptr(ys), _code(ys.dtype), _ptr(routing.row_of_pair), _ptr(out), n, ys.shape[1],
-          routing.top, _ptr(routing.weight) if routing.weights_on_output else None, _stream())
+          routing.top, _ptr(routing.weight) if routing.weights_on_output else None, _ptr(every),
+          _ptr(routing.side) if every is not None else None, _stream())
     return out
 
 

@@ -139,6 +139,7 @@ from . import niletar  # noqa: E402,F401
 from . import figonex  # noqa: E402,F401
 from . import giganex  # noqa: E402,F401
 from . import bolinex  # noqa: E402,F401
+from . import tabatar  # noqa: E402,F401
 
 
 def _import_plugins() -> None:

@@ -27,6 +27,10 @@ stream and from one kernel; what it hands on is the list of its outputs with the
 of two products: all that reads h is one matrix, all that is added to x another.  Then, where the layer has one, what it
 adds for the tokens themselves.
 
+``HyperConnectedBlock`` ("hyper_connected"): pre-norm sublayers between several residual streams, u = sum_s in_s X_s;
+y = sublayer(norm(u)); X_t <- sum_s mix[s, t] X_s + out_t y.  The residual it takes is a ``StreamSet`` and what it hands on
+a ``StreamMix``: the kernel that norms the next sublayer's input mixes the output in on the way.
+
 ``OutputNormBlock`` ("output_norm"): a norm on each sublayer's output only, x += norm1(mixer(x));
 x += norm2(feed_forward(x)); the sublayers read the stream itself.  What it hands on is a ``NormedDelta`` as well; the
 kernel that adds it also leaves the summed stream in the compute dtype for the sublayer that reads it next.
@@ -39,6 +43,7 @@ from ..kernels import ops
 from .linear import Linear
 from .norm import NormedDelta, StreamCopy
 from .registry import build_feed_forward, build_mixer, build_norm, register_block
+from .streams import HyperConnection, StreamMix, StreamSet
 from .token_side import TokenSide
 
 
@@ -272,7 +277,46 @@ class JointParallelBlock(Part):
         return super().kernel_libraries(dtype) + ["elementwise"]
 
 
+class HyperConnectedBlock(Part):
+    """``hyper_connected``: option ``streams``: how many; the connections are the parts ``hc1`` (mixer) and ``hc2``
+    (feed-forward).  A layer may have no feed-forward."""
+
+    def __init__(self, spec: BlockSpec) -> None:
+        super().__init__()
+        n_mixer_norm, n_mixer, n_ff_norm, n_ff = spec.names
+        streams = int(dict(spec.options)["streams"])
+        self.mixer_norm = self.add(n_mixer_norm, build_norm(spec.mixer_norm))
+        self.mixer = self.add(n_mixer, build_mixer(spec.mixer))
+        self.mixer_connection = self.add("hc1", HyperConnection(streams))
+        self.feed_forward = None
+        if spec.feed_forward is not None:
+            if spec.feed_forward_norm is None:
+                raise ValueError("a layer with a feed-forward needs its norm")
+            self.feed_forward_norm = self.add(n_ff_norm, build_norm(spec.feed_forward_norm))
+            self.feed_forward = self.add(n_ff, build_feed_forward(spec.feed_forward))
+            self.feed_forward_connection = self.add("hc2", HyperConnection(streams))
+        if not hasattr(self.mixer_norm, "apply_mixed"):
+            raise ValueError("a hyper_connected layer needs norms with apply_mixed (rmsnorm)")
+
+    def cache_request(self):
+        return self.mixer.cache_request()
+
+    def forward(self, residual, pending, batch, cache_view, writes_cache, dtype):
+        if not isinstance(residual, StreamSet):
+            raise ValueError("a hyper_connected layer needs the decoder's streams (DecoderSpec.streams)")
+        h = self.mixer_norm.apply_mixed(residual, pending, self.mixer_connection.w_in, dtype)
+        pending = StreamMix(self.mixer.forward(h, batch, cache_view, writes_cache), self.mixer_connection)
+        if self.feed_forward is None:
+            return pending
+        h = self.feed_forward_norm.apply_mixed(residual, pending, self.feed_forward_connection.w_in, dtype)
+        return StreamMix(self.feed_forward.forward(h), self.feed_forward_connection)
+
+    def kernel_libraries(self, dtype):
+        return super().kernel_libraries(dtype) + ["elementwise"]
+
+
 Block = PreNormBlock  # the name under which earlier callers know it
+register_block("hyper_connected", HyperConnectedBlock)
 register_block("parallel_joint", JointParallelBlock)
 register_block("parallel_residual", ParallelResidualBlock)
 register_block("output_norm", OutputNormBlock)

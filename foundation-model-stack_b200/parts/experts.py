@@ -22,10 +22,15 @@ Further options, each of which leaves the above as it is when absent:
                               equal groups of neighbours of which the ``keep`` best can be chosen from (a group's score:
                               the sum of its two largest choice scores); the weights are the chosen s as they are, times
                               ``route_scale``, and multiply the experts' OUTPUTS
+    ``scoring`` "softmax_chosen"  the ``top`` largest logits Wr h + ``router_bias`` (a vector of the checkpoint, where
+                              ``router_bias`` is set) are a token's experts, its weights the softmax over those logits
+                              alone, times ``route_scale``; they multiply the experts' OUTPUTS
     ``unit`` "relu_squared"   expert_e(v) = Wdown,e relu(Wup,e v)^2: no gate; ``up`` [experts, hidden, dim]
     ``unit`` "silu"           expert_e(v) = Wdown,e (silu(Wgate,e v) * Wup,e v)
-    ``shared`` spec           a further unit that runs for every token, a ``projected_unit`` whose products the block makes
-                              with its mixer's
+    ``shared`` spec           a further unit that runs for every token: a ``projected_unit``, whose products the block makes
+                              with its mixer's, or a feed-forward of its own, whose output is added here
+    ``shared_gate``           the latter's output is multiplied by sigmoid(w h), one number a token; w is the row of the
+                              router's matrix behind the experts' rows (the router's product makes both)
 """
 from __future__ import annotations
 
@@ -39,6 +44,9 @@ from .registry import build_feed_forward, register_feed_forward
 
 
 class RoutedExperts(Part):
+    _ROUTE_MODES = {"sigmoid": ops.ROUTE_SIGMOID, "softmax": ops.ROUTE_SOFTMAX, "sigmoid_groups": ops.ROUTE_SIGMOID_GROUPS,
+                    "softmax_chosen": ops.ROUTE_SOFTMAX_CHOSEN}
+
     def __init__(self, spec: FeedForwardSpec) -> None:
         super().__init__()
         o = dict(spec.options)
@@ -48,8 +56,7 @@ class RoutedExperts(Part):
         if not (0 < self.top <= self.experts) or self.hidden <= 0:
             raise ValueError(f"routed_experts: {self.experts} experts, top {self.top}, hidden {self.hidden}")
         self.scoring, self.unit = o.get("scoring", "sigmoid"), o.get("unit", "gated_clamped")
-        if (self.scoring not in ("sigmoid", "softmax", "sigmoid_groups")
-                or self.unit not in ("gated_clamped", "relu_squared", "silu")):
+        if self.scoring not in self._ROUTE_MODES or self.unit not in ("gated_clamped", "relu_squared", "silu"):
             raise ValueError(f"routed_experts: scoring {self.scoring!r}, unit {self.unit!r}")
         if self.unit == "gated_clamped" and "limit" not in o:
             raise ValueError("routed_experts: the gated unit needs its limit")
@@ -60,10 +67,19 @@ class RoutedExperts(Part):
             raise ValueError(f"routed_experts: {self.experts} experts in {self.groups} groups of which {self.keep} stay, "
                              f"top {self.top}")
         shared = build_feed_forward(o["shared"]) if o.get("shared") is not None else None
+        self.shared = None
+        if shared is not None and not hasattr(shared, "in_rows"):  # a feed-forward with products of its own
+            self.shared, shared = self.add("shared", shared), None
+        self.shared_gate = bool(o.get("shared_gate", False))
+        if self.shared_gate and self.shared is None:
+            raise ValueError("routed_experts: a gate without a shared unit of its own")
         self.in_rows = shared.in_rows if shared else 0
         self.joint_hidden, self.activation = (shared.hidden, shared.activation) if shared else (0, 0)
         self.gated = shared.gated if shared else False
-        self.router = self.add("router", Linear(spec.dim, self.experts, False))
+        self.router = self.add("router", Linear(spec.dim, self.experts + (1 if self.shared_gate else 0), False))
+        self.has_bias = bool(o.get("router_bias", False))
+        if self.has_bias:
+            self.declare("router_bias", (self.experts,), role="vector")
         if self.has_correction:
             self.declare("correction", (self.experts,), role="vector")
         if self.unit == "relu_squared":
@@ -71,12 +87,14 @@ class RoutedExperts(Part):
         else:
             self.declare("gate_up", (self.experts, 2 * self.hidden, spec.dim), role="matrix")
         self.declare("down", (self.experts, spec.dim, self.hidden), role="matrix")
-        self._correction = None
+        self._correction = self._bias = None
 
     def finalize(self, device, dtype) -> None:
         super().finalize(device, dtype)
         if self.has_correction:
             self._correction = self.tensor("correction").float().contiguous()
+        if self.has_bias:
+            self._bias = self.tensor("router_bias").float().contiguous()
 
     def beside(self, x):
         """What a block that makes its sublayers' products together adds as it is: the routed experts."""
@@ -88,23 +106,23 @@ class RoutedExperts(Part):
         return self._routed(x)
 
     def _routed(self, x):
-        if self.scoring == "sigmoid_groups":
-            routing = ops.route(x, self.router.tensor("weight"), self.top, ops.ROUTE_SIGMOID_GROUPS, self._correction,
-                                self.route_scale, self.groups, self.keep)
-        elif self.scoring == "softmax":
-            routing = ops.route(x, self.router.tensor("weight"), self.top, ops.ROUTE_SOFTMAX, self._correction,
-                                self.route_scale)
+        every = self.shared.forward(x) if self.shared is not None else None
+        mode, further = self._ROUTE_MODES[self.scoring], {"bias": self._bias, "side": self.shared_gate}
+        if self.scoring == "sigmoid":
+            routing = ops.route(x, self.router.tensor("weight"), self.top, mode, **further)
         else:
-            routing = ops.route(x, self.router.tensor("weight"), self.top)
+            routing = ops.route(x, self.router.tensor("weight"), self.top, mode, self._correction, self.route_scale, self.groups,
+                                self.keep, **further)
         if self.unit == "relu_squared":
             hidden = ops.routed_linear(routing.rows, self.tensor("up"), routing, relu_squared=True)
-            return ops.route_gather(ops.routed_linear(hidden, self.tensor("down"), routing), routing)
+            return ops.route_gather(ops.routed_linear(hidden, self.tensor("down"), routing), routing, every)
         hidden = ops.routed_linear(routing.rows, self.tensor("gate_up"), routing, True, self.limit, self.alpha,
                                    silu=self.unit == "silu")
-        return ops.route_gather(ops.routed_linear(hidden, self.tensor("down"), routing), routing)
+        return ops.route_gather(ops.routed_linear(hidden, self.tensor("down"), routing), routing, every)
 
     def kernel_libraries(self, dtype):
-        return ["grouped", "elementwise"] + (["gemm_bf16_skinny"] if dtype == torch.bfloat16 else [])
+        own = self.shared.kernel_libraries(dtype) if self.shared is not None else []
+        return own + ["grouped", "elementwise"] + (["gemm_bf16_skinny"] if dtype == torch.bfloat16 else [])
 
 
 register_feed_forward("routed_experts", RoutedExperts)

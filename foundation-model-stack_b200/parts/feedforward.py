@@ -1,6 +1,8 @@
 """Feed-forwards.  ``GatedLinearUnit``: y = W2 (act(Wg x) * (W1 x)) with the gate and up rows fused into
 one matrix, gate first (fms/modules/feedforward.py:227-240 for the sizes, :288-297 for the formula).
 
+``PlainUnit`` ("mlp"): y = W2 act(W1 x), ungated.
+
 Interface of a feed-forward (what a block calls):
 
     forward(x) -> y          x, y: [tokens, dim] in the compute dtype
@@ -46,6 +48,23 @@ class GatedLinearUnit(Part):
         return super().kernel_libraries(dtype) + ["elementwise"]
 
 
+class PlainUnit(Part):
+    def __init__(self, spec: FeedForwardSpec) -> None:
+        super().__init__()
+        act = spec.activation.lower()
+        if act not in UNGATED_ACTIVATIONS:
+            raise ValueError(f"activation {spec.activation!r} is not supported; supported: {sorted(UNGATED_ACTIVATIONS)}")
+        self.activation = UNGATED_ACTIVATIONS[act]
+        self.up = self.add("w1", Linear(spec.dim, spec.hidden, spec.bias))
+        self.down = self.add("w2", Linear(spec.hidden, spec.dim, spec.bias))
+
+    def forward(self, x):
+        return self.down.forward(ops.activated_linear(x, self.up.tensor("weight"), self.up.tensor("bias"), self.activation))
+
+    def kernel_libraries(self, dtype):
+        return super().kernel_libraries(dtype) + ["elementwise"]
+
+
 class ProjectedUnit(Part):
     def __init__(self, spec: FeedForwardSpec) -> None:
         super().__init__()
@@ -64,4 +83,5 @@ class ProjectedUnit(Part):
 
 
 register_feed_forward("glu", GatedLinearUnit)
+register_feed_forward("mlp", PlainUnit)
 register_feed_forward("projected_unit", ProjectedUnit)

@@ -17,6 +17,15 @@ queries of ``head_dim``, values of ``vdim``, all laid out head by head:
     o_t = S_t^T q / (max(|n_t . q|, exp(-m_t)) + 1e-6)
     out = Wo (o / rms(o) * w * sigmoid(Wg h))                                 the root mean square per head; w [H * vdim]
 
+``GatedLinearAttention`` ("gla"): one decay a key channel, from a low-rank product,
+
+    q = Wq h / sqrt(head_dim), k = Wk h, v = Wv h
+    a = sigmoid(Wa2 (Wa1 h) + ba2)^(1 / tau)                                               per head and key channel
+    S_t = diag(a_t) S_(t-1) + k_t v_t^T;  o_t = S_t^T q_t
+    out = Wo (o / rms(o) * w * silu(Wg h))                                    the root mean square per head; w [vdim], shared
+
+Its fused projection is [q; k; v; g; a1] and Wa2 a product inside the kernel that makes q, k, v and the decays ready.
+
 Everything that reads h is one fused projection, [q; k; v; g] or [q; k; v; g; i; f], its rows filled up with zeros to a
 multiple of 8; the gates' biases are added in float32 by the kernel that takes the gates.  Per sequence the cache holds
 the state matrices in float32 ([heads, vdim, head_dim], a column's rows contiguous) and, for the gated form, the
@@ -43,6 +52,7 @@ class _DecayedStateMixer(Part):
     """What the two kinds share: sizes, the fused projection, the output norm's weight, the output projection."""
 
     extra_rows_per_head = 0  # rows of the fused projection behind [q; k; v; g], per head
+    norm_per_head = False  # the output norm's weight: one for all heads together, or one of a head's size for each
 
     def __init__(self, spec: MixerSpec) -> None:
         super().__init__()
@@ -53,15 +63,21 @@ class _DecayedStateMixer(Part):
             raise ValueError(f"{spec.kind}: {self.heads} heads of {self.head_dim} (up to 256) with values of {self.vdim}")
         self.inner = self.heads * self.vdim
         self.gate_col = self.heads * (2 * self.head_dim + self.vdim)  # where [g] starts in the fused projection's rows
-        self.in_proj = self.add("in_proj", Linear(spec.dim, self.fused_rows(self.heads, self.head_dim, self.vdim), False))
-        self.declare("norm", (self.inner,), role="vector")
+        self.in_proj = self.add("in_proj", Linear(spec.dim, self.fused_rows(self.heads, self.head_dim, self.vdim,
+                                                                            self.extra_rows(o)), False))
+        self.declare("norm", (self.vdim if self.norm_per_head else self.inner,), role="vector")
         self.dense = self.add("dense", Linear(self.inner, spec.dim, False))
         self._norm = None
 
+    @staticmethod
+    def extra_rows(options: dict) -> int:
+        """Rows of the fused projection behind everything that goes by heads."""
+        return 0
+
     @classmethod
-    def fused_rows(cls, heads: int, head_dim: int, vdim: int) -> int:
+    def fused_rows(cls, heads: int, head_dim: int, vdim: int, extra: int = 0) -> int:
         """Rows of the fused projection: what a checkpoint adapter has to put together."""
-        return _round8(heads * (2 * head_dim + 2 * vdim + cls.extra_rows_per_head))
+        return _round8(heads * (2 * head_dim + 2 * vdim + cls.extra_rows_per_head) + extra)
 
     def finalize(self, device, dtype) -> None:
         super().finalize(device, dtype)
@@ -126,5 +142,38 @@ class MatrixLSTM(_DecayedStateMixer):
         return self.dense.forward(y)
 
 
+class GatedLinearAttention(_DecayedStateMixer):
+    norm_per_head = True
+
+    @staticmethod
+    def extra_rows(options: dict) -> int:
+        return int(options["rank"])
+
+    def __init__(self, spec: MixerSpec) -> None:
+        super().__init__(spec)
+        o = dict(spec.options)
+        self.rank, self.tau = int(o["rank"]), float(o["tau"])
+        if self.rank <= 0 or not self.tau > 0.0:
+            raise ValueError(f"gla: rank {self.rank}, tau {self.tau}")
+        self.rank_col = self.gate_col + self.inner
+        self.decay_out = self.add("decay_out", Linear(self.rank, self.heads * self.head_dim, True))
+        self._decay_bias = None
+
+    def finalize(self, device, dtype) -> None:
+        super().finalize(device, dtype)
+        self._decay_bias = self.decay_out.tensor("bias").float().contiguous()
+
+    def cache_request(self):
+        return StateRequest((self.heads, self.vdim, self.head_dim), torch.float32, "state_matrix")
+
+    def forward(self, x, batch, cache_view, writes_cache: bool = True):
+        proj = self.in_proj.forward(x)
+        o = ops.gla_scan(proj, cache_view.state, batch, self.heads, self.head_dim, self.vdim, self.rank_col,
+                         self.decay_out.tensor("weight"), self._decay_bias, self.tau, self.head_dim ** -0.5, writes_cache)
+        y = ops.gated_group_rmsnorm(o, proj, self.gate_col, ops.GATE_SILU_AFTER, self._norm, self.eps, self.vdim, proj.dtype)
+        return self.dense.forward(y)
+
+
+register_mixer("gla", GatedLinearAttention)
 register_mixer("lightning_attention", LightningAttention)
 register_mixer("mlstm", MatrixLSTM)

@@ -23,6 +23,9 @@ by value.
 the weight; adds several pending outputs with a factor each; ``apply_pair`` gives two norms of the same stream from
 one kernel.
 
+``apply_mixed`` (``RMSNorm``): the same for a token with several residual streams (``StreamSet``): the pending output is
+mixed into all of them and the norm is of their weighted sum; ``apply`` on a ``StreamSet`` norms their plain sum.
+
 ``LayerNorm`` ("layernorm"): y = (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * w.  Option ``bias``: + b (a vector
 of the checkpoint; the norm of the stream only).  Option
 ``layer_scale``: a second vector ``scale`` multiplies the result element by element (the gain the kernel sees is
@@ -38,6 +41,7 @@ from ..config.specs import NormSpec
 from ..kernels import ops
 from .base import Part
 from .registry import register_norm
+from .streams import StreamMix, StreamSet
 
 
 class NormedDelta:
@@ -72,13 +76,13 @@ class RMSNorm(Part):
         self.eps = float(spec.eps)
         self.offset = float(dict(spec.options).get("offset", 0.0))
         self.declare("weight", (spec.dim,), role="vector")
-        self._gain = self._wide_gain = None
+        self._gain = self._wide_gain = self._ones = None
 
     def finalize(self, device, dtype) -> None:
         super().finalize(device, dtype)
         if self.offset != 0.0:
             self._gain = (self.tensor("weight").float() + self.offset).contiguous()
-        self._wide_gain = None
+        self._wide_gain = self._ones = None
 
     def mode_and_gain(self):
         """(mode, float32 gain vector, eps): what ``ops.normed_add_norm`` takes."""
@@ -93,7 +97,20 @@ class RMSNorm(Part):
         """(vector or None, the one number where there is no vector, eps): what the fused kernel takes."""
         return self.gain_vector(), 1.0, self.eps
 
+    def apply_mixed(self, streams, pending, w_in, out_dtype, rows=None):
+        """norm(sum_s w_in[s] X_s) of a ``StreamSet``, after what is pending (a ``StreamMix`` or None) has gone into the
+        streams.  With ``rows`` only those tokens are computed and the streams stay as they are."""
+        if pending is not None and not isinstance(pending, StreamMix):
+            raise ValueError("several residual streams take a pending output with the weights that mix it in (StreamMix)")
+        _, gain, eps = self.mode_and_gain()
+        delta, on = (pending.delta, pending.connection.on) if pending is not None else (None, None)
+        return ops.stream_mix_norm(streams, delta, on, w_in, gain, eps, out_dtype, rows)
+
     def apply(self, residual, delta, out_dtype, rows=None):
+        if isinstance(residual, StreamSet):
+            if self._ones is None:
+                self._ones = torch.ones(residual.streams, dtype=torch.float32, device=residual.start.device)
+            return self.apply_mixed(residual, delta, self._ones, out_dtype, rows)
         if isinstance(delta, StreamCopy):
             delta = None
         if isinstance(delta, NormedDelta):
