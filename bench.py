@@ -1112,6 +1112,125 @@ def run_bolinex(args):
 
 
 # --------------------------------------------------------------------------------------------------
+# --compare tabatar: the Tabatar design beside Llama at equal width, layer for layer
+# --------------------------------------------------------------------------------------------------
+TABATAR_SHAPE = dict(width=4096, vocab=128256, streams=2, ff=14336, experts=16, top=4, expert_ff=3584, shared_ff=3584, heads=32,
+                     kv_heads=8, dim=128, vdim=128, window=4096, gla_heads=32, gla_dim=128, gla_vdim=128, tau=16.0, rank=16,
+                     softcap=30.0)
+
+
+def tabatar_layers(kinds, mlps):
+    """`kinds`: the mixers ("attention", "gla"), `mlps`: their feed-forwards ("dense", "moe", None)."""
+    from fms_b200.models.tabatar import attention_layer, dense_mlp, gla_layer, moe_mlp
+
+    g = TABATAR_SHAPE
+    rot = {"base": 500000.0, "dims": g["dim"], "scaling": {"factor": 8.0, "high": 4.0, "low": 1.0, "original": 8192}}
+    out = []
+    for kind, which in zip(kinds, mlps):
+        mlp = {None: lambda: None, "dense": lambda: dense_mlp(g["ff"]),
+               "moe": lambda: moe_mlp(g["experts"], g["top"], g["expert_ff"], g["shared_ff"])}[which]()
+        out.append(attention_layer(g["heads"], g["kv_heads"], g["dim"], g["vdim"], g["dim"] ** -0.5, g["window"], rot, mlp)
+                   if kind == "attention" else gla_layer(g["gla_heads"], g["gla_dim"], g["gla_vdim"], g["tau"], g["rank"], mlp))
+    return out
+
+
+def tabatar_counts(layers, tokens, batch_context, batch):
+    """(flops of a prompt of `tokens`, bytes a decode step of `batch` sequences with `batch_context` cached tokens
+    reads and writes) of the given layers: products, attention over the cache, the matrix memories (6 flops per state value
+    and token, float32 on the CUDA cores; the states read and written once a step), the experts each token uses (for a
+    decode step: the distinct experts that `batch` tokens are expected to hit)."""
+    g = TABATAR_SHAPE
+    d, flops, moved = g["width"], 0.0, 0.0
+    for layer in layers:
+        m = layer["mixer"]
+        h, k, v = m["heads"], m["dim"], m["vdim"]
+        if layer["type"] == "attention":
+            kv = m["kv_heads"]
+            w = d * (h * k + kv * (k + v) + h * v) + h * v * d
+            flops += tokens * tokens * h * (k + v)  # the causal half of 2 T^2 (dim + vdim) a head
+            moved += 2 * batch_context * kv * (k + v)
+        else:
+            w = d * (2 * h * k + 2 * h * v + m["rank"]) + m["rank"] * h * k + h * v * d
+            flops += 6.0 * tokens * h * k * v
+            moved += 2 * 4 * batch * h * k * v
+        mlp = layer.get("mlp")
+        if mlp and mlp["kind"] == "dense":
+            w += 2 * mlp["ff"] * d
+        elif mlp:
+            e, top, f = mlp["router"]["experts"], mlp["router"]["top"], mlp["expert"]["ff"]
+            w += 3 * mlp["shared"]["ff"] * d + (e + 1) * d
+            flops += 2.0 * tokens * top * 3 * f * d
+            moved += 2 * e * (1 - (1 - top / e) ** batch) * 3 * f * d
+        flops += 2.0 * tokens * w
+        moved += 2 * w
+    head = 2 * g["vocab"] * d
+    return flops + head, moved + head
+
+
+class TabatarMeasured(Measured):
+    """A Tabatar model of given layers on the device, measured like the Llama one."""
+
+    def __init__(self, layers, room, max_prompt, slots):
+        import torch
+
+        from fms_b200.models.tabatar import Tabatar, TabatarConfig
+        from fms_b200.weights.sources import RandomSource
+
+        g = TABATAR_SHAPE
+        self.m, self.dtype, self.nlayers, self.itemsize, self.layers = dict(vocab=g["vocab"]), "bf16", len(layers), 2, layers
+        self.model = Tabatar(TabatarConfig(vocab=g["vocab"], width=g["width"], embedding_scale=g["width"] ** 0.5, streams=g["streams"],
+                                           logit_softcap=g["softcap"], layers=layers))
+        self.model.load(RandomSource(self.model.checkpoint_layout(), 0, dtype=torch.bfloat16, device="cuda"), "native", "cuda",
+                        torch.bfloat16)
+        self.engine = self.model.new_engine(max_tokens=slots * (max_prompt + 2 * room + 128), max_slots=slots)
+        self.torch = torch
+
+
+def run_tabatar(args):
+    """One JSON line: prompts of 512 and 2,048 tokens and decode steps of 1, 8 and 64 sequences, for `--layers` layers
+    (default 4) of the Tabatar design at the width of the benchmark's Llama (attention with the dense feed-forward of 14,336
+    and gated linear attention of 32 heads of 128 x 128 with 16 experts of 3,584 of which a token takes 4, beside a shared one,
+    taking turns, between two residual streams), for as many Llama-3-8B layers, for each mixer alone, and for each
+    feed-forward under attention.  Each figure with its fraction of the measured peak: flops of a prompt over the bf16
+    product peak, bytes a decode step moves over the copy peak."""
+    pk = peaks()
+    n = args.layers or 4
+    steps, warm = max(16, args.steps // 2), max(3, args.warmup // 2)
+    room = warm + 3 * steps + 8
+    lengths = {1: [1024], 8: [1024] * 8, 64: [1024] * 64}
+    out = {"compare": "tabatar", "layers": n, "shape": TABATAR_SHAPE, "peaks": pk, "steps": steps, "warmup": warm, "models": {}}
+
+    def measure(run, name, flops_bytes):
+        row = {}
+        for tokens in (512, 2048):
+            ms = run.prefill(tokens, 3)
+            row[f"prefill_{tokens}"] = {"ms": round(ms, 3), "tok_s": round(tokens / (ms / 1e3), 1),
+                                        "frac_of_bf16_peak": round(flops_bytes(tokens, 0, 0)[0] / (ms / 1e3) / 1e12 / pk["bf16_tflops"], 4)}
+        for b in (1, 8, 64):
+            v, ms, ctx, _, _ = run.device_decode(b, steps, warm, lengths[b], regions=3)
+            row[f"decode_b{b}"] = {"ms": round(ms, 4), "tok_s": round(v, 1),
+                                   "frac_of_copy_peak": round(flops_bytes(0, ctx, b)[1] / (ms / 1e3) / 1e9 / pk["hbm_gbs"], 4)}
+        out["models"][name] = row
+        run.close()
+
+    mixed = [("attention", "dense"), ("gla", "moe")]
+    variants = [("tabatar", tabatar_layers([mixed[i % 2][0] for i in range(n)], [mixed[i % 2][1] for i in range(n)])),
+                ("attention_only", tabatar_layers(["attention"] * n, [None] * n)),
+                ("gla_only", tabatar_layers(["gla"] * n, [None] * n)),
+                ("attention_with_dense", tabatar_layers(["attention"] * n, ["dense"] * n)),
+                ("attention_with_experts", tabatar_layers(["attention"] * n, ["moe"] * n))]
+    if args.only:
+        variants = [v for v in variants if v[0] == args.only]
+    for name, layers in variants:
+        measure(TabatarMeasured(layers, room, 2048, 64), name,
+                lambda tokens, ctx, b, layers=layers: tabatar_counts(layers, tokens, ctx, b))
+    if not args.only or args.only == "llama":
+        llama = Measured(MODEL, "bf16", n, room, 2048, slots=64)
+        measure(llama, "llama", lambda tokens, ctx, b: (prefill_flops(n, tokens), decode_bytes(n, ctx)))
+    print(json.dumps(out))
+
+
+# --------------------------------------------------------------------------------------------------
 def main():
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
     ap.add_argument("--gpus", type=int, default=int(os.environ.get("WORLD_SIZE", "1")))
@@ -1128,7 +1247,7 @@ def main():
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS, help="with --only prefill: the prompt's length")
     ap.add_argument("--points", choices=["default", "main", "long"], default="default",
                     help="main: without the further configurations; long: also decode at batch 64 with 8k contexts")
-    ap.add_argument("--compare", choices=["", "goletar", "niletar", "figonex", "giganex", "bolinex"], default="",
+    ap.add_argument("--compare", choices=["", "goletar", "niletar", "figonex", "giganex", "bolinex", "tabatar"], default="",
                     help="goletar: the Goletar design beside as many Llama layers of equal width (--layers, default 4; "
                     "--only goletar|mingru_only|latent_attention_only|mingru_with_experts|llama for one of them); "
                     "niletar: the Niletar design likewise (--only niletar|parallel_only|mamba2_only|llama); "
@@ -1136,6 +1255,8 @@ def main():
                     "giganex: the Giganex design likewise (--only giganex|parallel_only|latent_attention_only|attention_only|"
                     "attention_with_experts|llama); "
                     "bolinex: the Bolinex design likewise (--only bolinex|attention_only|attention_with_dense|"
+                    "attention_with_experts|llama); "
+                    "tabatar: the Tabatar design likewise (--only tabatar|attention_only|gla_only|attention_with_dense|"
                     "attention_with_experts|llama)")
     args = ap.parse_args()
     choose_model(args.model)
@@ -1153,6 +1274,8 @@ def main():
         run_giganex(args)
     elif args.compare == "bolinex":
         run_bolinex(args)
+    elif args.compare == "tabatar":
+        run_tabatar(args)
     elif args.impl == "reference":
         run_reference(args)
     elif args.only in ("gemm_rows", "attention_prefill", "attention_decode"):

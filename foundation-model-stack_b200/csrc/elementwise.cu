@@ -1197,6 +1197,7 @@ FMS_API int fms_parts_group_rmsnorm(float* residual, const void* d0, float s0, c
 //         plain rotation: stretched frequencies come with such a constant)
 //   q, k: x / sqrt(mean(x^2) + eps) over the head's dim values, where qk_norm is set (no gain)
 //         (`norm_first`: the norm comes before the rotation, times q_gain / k_gain [dim] where those are given)
+//   `sincos` [tokens, rot / 2]: the (sin, cos) of every token's angles where the step has made that table already
 //   `v_from_k`: there are no value columns; the value is the key as projected, before norm and rotation
 //   `v_first`: value c of a token becomes (1 - v_mix) v + v_mix v_first[t, c], mixed in float32 (the values of an
 //         earlier layer, columns of another matrix with row stride first_stride)
@@ -1214,7 +1215,8 @@ __global__ void qk_prepare_store_kernel(const T* proj, int stride, T* q_out, con
                                         const int* token_seq, const int* slots, T* k_cache, T* v_cache, const int* table,
                                         int table_stride, int block_tokens, int nheads, int kvheads, int dim, int vdim,
                                         int pad, int write_cache, int* error_flag, int n_seqs, int table_rows,
-                                        int pool_blocks, const T* v_first, int first_stride, float v_mix, int vec) {
+                                        int pool_blocks, const T* v_first, int first_stride, float v_mix, const float2* sincos,
+                                        int vec) {
   __shared__ float2 sc[PREP_MAX_PAIRS];
   pdl_launch_dependents();
   pdl_wait();
@@ -1223,7 +1225,12 @@ __global__ void qk_prepare_store_kernel(const T* proj, int stride, T* q_out, con
   const int pid = position_ids ? __ldcg(position_ids + t) : pos;
   for (int i = threadIdx.x; i < rot / 2; i += blockDim.x) {
     float s, c;
-    sincosf((float)pid * inv_freq[i], &s, &c);
+    if (sincos) {
+      const float2 v = sincos[(size_t)t * (rot / 2) + i];
+      s = v.x, c = v.y;
+    } else {
+      sincosf((float)pid * inv_freq[i], &s, &c);
+    }
     sc[i] = make_float2(s * rot_mult, c * rot_mult);
   }
   __syncthreads();
@@ -1296,6 +1303,43 @@ __global__ void qk_prepare_store_kernel(const T* proj, int stride, T* q_out, con
       // the norm (with its gain, where there is one) comes first and the rotation turns the normed values
       const float* gain = is_q ? q_gain : k_gain;
       float ss = 0.f;
+      if (vec && halves && half % 4 == 0) {  // four neighbours a lane (the gains are vectors of the model: 16-byte aligned)
+        for (int e = 4 * lane; e < dim; e += 128) {
+          float x[4];
+          ldv4(src + e, x);
+#pragma unroll
+          for (int k = 0; k < 4; ++k) ss += x[k] * x[k];
+        }
+        const float inv = qk_norm ? 1.f / sqrtf(warp_sum(ss) / (float)dim + eps) : 1.f;
+        for (int i = 4 * lane; i < half; i += 128) {
+          float x0[4], x1[4], g0[4] = {1.f, 1.f, 1.f, 1.f}, g1[4] = {1.f, 1.f, 1.f, 1.f};
+          ldv4(src + i, x0);
+          ldv4(src + half + i, x1);
+          if (gain) {
+            ldv4(gain + i, g0);
+            ldv4(gain + half + i, g1);
+          }
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const float a = x0[k] * inv * g0[k], b = x1[k] * inv * g1[k];
+            x0[k] = sc[i + k].y * a - sc[i + k].x * b;
+            x1[k] = sc[i + k].y * b + sc[i + k].x * a;
+          }
+          stv4(dst + i, x0);
+          stv4(dst + half + i, x1);
+        }
+        for (int e = rot + 4 * lane; e < pad; e += 128) {
+          float x[4] = {0.f, 0.f, 0.f, 0.f}, g[4] = {1.f, 1.f, 1.f, 1.f};
+          if (e < dim) {
+            ldv4(src + e, x);
+            if (gain) ldv4(gain + e, g);
+          }
+#pragma unroll
+          for (int k = 0; k < 4; ++k) x[k] = x[k] * inv * g[k];
+          stv4(dst + e, x);
+        }
+        return;
+      }
       for (int e = lane; e < dim; e += 32) {
         const float x = to_f32(src[e]);
         ss += x * x;
@@ -1339,7 +1383,8 @@ FMS_API int fms_qk_prepare_store(const void* proj, int dtype, int stride, void* 
                                  const int* token_seq, const int* slots, void* k_cache, void* v_cache, const int* table,
                                  int table_stride, int block_tokens, int n_tokens, int nheads, int kvheads, int dim,
                                  int vdim, int pad, int write_cache, int* error_flag, int n_seqs, int table_rows,
-                                 int pool_blocks, const void* v_first, int first_stride, float v_mix, cudaStream_t stream) {
+                                 int pool_blocks, const void* v_first, int first_stride, float v_mix, const void* sincos,
+                                 cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (v_first && v_from_k) return fms_fail("qk_prepare_store: values that are the keys are not mixed with others");
   if (rot < 0 || rot % 2 || rot > dim || rot / 2 > PREP_MAX_PAIRS || (rot > 0 && inv_freq == nullptr))
@@ -1350,7 +1395,8 @@ FMS_API int fms_qk_prepare_store(const void* proj, int dtype, int stride, void* 
   const size_t item = dtype == FMS_BF16 ? 2 : 4;
   const int vec = dim % 4 == 0 && vdim % 4 == 0 && pad % 4 == 0 && stride % 4 == 0 && first_stride % 4 == 0 &&
                   (uintptr_t)proj % (4 * item) == 0 && (uintptr_t)q_out % (4 * item) == 0 && (uintptr_t)k_cache % (4 * item) == 0 &&
-                  (uintptr_t)v_cache % (4 * item) == 0 && (uintptr_t)v_first % (4 * item) == 0;
+                  (uintptr_t)v_cache % (4 * item) == 0 && (uintptr_t)v_first % (4 * item) == 0 && (uintptr_t)q_gain % 16 == 0 &&
+                  (uintptr_t)k_gain % 16 == 0;
   const int items = (q_out ? nheads : 0) + 2 * kvheads;
   FMS_DISPATCH_DTYPE(dtype, T,
                      fms_launch(qk_prepare_store_kernel<T>, dim3(n_tokens, (items + 3) / 4), dim3(128), 0, stream,
@@ -1359,7 +1405,7 @@ FMS_API int fms_qk_prepare_store(const void* proj, int dtype, int stride, void* 
                                 positions, position_ids, token_seq, slots,
                                 (T*)k_cache, (T*)v_cache, table, table_stride, block_tokens, nheads, kvheads, dim, vdim, pad,
                                 write_cache, error_flag, n_seqs, table_rows, pool_blocks, (const T*)v_first, first_stride, v_mix,
-                                vec));
+                                (const float2*)sincos, vec));
   return fms_launch_status("qk_prepare_store");
 }
 

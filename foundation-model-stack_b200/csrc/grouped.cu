@@ -468,14 +468,14 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(const T* x, con
 __global__ void __launch_bounds__(32 * CHOOSE_WARPS) route_choose_kernel(const float* logits, int* expert, float* weight, int n_tokens,
                                                                          int experts, int top, int mode, const float* correction,
                                                                          float route_scale, int groups, int keep,
-                                                                         const float* bias, float* side) {
+                                                                         const float* bias, float* side, int logit_stride) {
   extern __shared__ float sm[];  // a warp: `experts` logits, `experts` scores, `groups` scores
   pdl_launch_dependents();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * CHOOSE_WARPS + warp;
   if (t >= n_tokens) return;
   float* logit = sm + (size_t)warp * (2 * experts + groups);
-  const float* mine = logits + (size_t)t * (experts + (side ? 1 : 0));
+  const float* mine = logits + (size_t)t * logit_stride;
   for (int e = lane; e < experts; e += 32) logit[e] = bias ? mine[e] + bias[e] : mine[e];
   if (side && lane == 0) side[t] = 1.f / (1.f + expf(-mine[experts]));
   __syncwarp();
@@ -660,13 +660,13 @@ FMS_API int fms_grouped_linear(const void* x, const void* w, void* y, int dtype,
 // choice by score + correction among the experts of the `keep` best of `groups` equal groups of neighbours (a group's
 // score: the sum of its two largest choice scores), weights the chosen scores times route_scale; rows as in mode 1.
 // mode 3: the choice is by logit, weights the softmax over the chosen logits only, times route_scale; rows as in mode 1.
-// logits: [n_tokens, rows of router] float32 = x . router^T where the caller has them already, else null.
+// logits: rows of logit_stride float32, the first of which are x . router^T, where the caller has them already, else null.
 // bias: [experts] float32 that is added to the logits first, or null.  side: [n_tokens] float32, or null: the router then has
 // a row behind the experts' and side[t] = sigmoid(x[t] . that row), the gate of a unit that every token uses.
 FMS_API int fms_route(const void* x, int dtype, const void* router, int router_dtype, int* expert, float* weight, int* counts,
                       int* offsets, int* tile_first, int* row_of_pair, int* group_of_row, void* xs, int n_tokens, int dim,
                       int experts, int top, int mode, const float* correction, float route_scale, int groups, int keep,
-                      const float* logits, const float* bias, float* side, cudaStream_t stream) {
+                      const float* logits, int logit_stride, const float* bias, float* side, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (dim <= 0 || experts <= 0 || top <= 0 || top > experts) return fms_fail("route: dim %d, experts %d, top %d", dim, experts, top);
   if (mode < 0 || mode > 3) return fms_fail("route: mode %d", mode);
@@ -677,7 +677,8 @@ FMS_API int fms_route(const void* x, int dtype, const void* router, int router_d
   if (logits != nullptr) {
     if (CHOOSE_WARPS * choice > 48 * 1024) return fms_fail("route: %d experts in %d groups do not fit shared memory", experts, groups);
     fms_launch(route_choose_kernel, dim3((n_tokens + CHOOSE_WARPS - 1) / CHOOSE_WARPS), dim3(32 * CHOOSE_WARPS), CHOOSE_WARPS * choice,
-               stream, logits, expert, weight, n_tokens, experts, top, mode, correction, route_scale, groups, keep, bias, side);
+               stream, logits, expert, weight, n_tokens, experts, top, mode, correction, route_scale, groups, keep, bias, side,
+               logit_stride);
   } else {
     const size_t smem = (size_t)dim * sizeof(float) + choice;
     if (smem > 200 * 1024) return fms_fail("route: rows of %d values and %d experts do not fit shared memory", dim, experts);

@@ -64,7 +64,7 @@ _SIGNATURES = {
     "fms_normed_add_rmsnorm": [_P, _P, _I, _P, _F, _F, _P, _F, _F, _I, _P, _I, _P, _I, _I, _I, _P],
     "fms_mingru_scan": [_P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _P, _P, _I, _P, _P],
     "fms_grouped_linear": [_P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _L, _L, _L, _L, _I, _F, _F, _I, _P],
-    "fms_route": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _F, _I, _I, _P, _P, _P, _P],
+    "fms_route": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _F, _I, _I, _P, _I, _P, _P, _P],
     "fms_route_gather": [_P, _I, _P, _P, _I, _I, _I, _P, _P, _P, _P],
     "fms_relu_squared": [_P, _I, _L, _P],
     "fms_gated_clamped": [_P, _P, _I, _I, _I, _F, _F, _P],
@@ -79,13 +79,14 @@ _SIGNATURES = {
     "fms_cast_rows": [_P, _P, _I, _L, _P],
     "fms_parts_group_rmsnorm": [_P, _P, _F, _P, _F, _P, _F, _P, _F, _P, _P, _F, _I, _P, _P, _I, _P, _I, _I, _I, _P],
     "fms_qk_prepare_store": [_P, _I, _I, _P, _P, _I, _F, _I, _F, _P, _P, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I,
-                             _I, _I, _I, _I, _I, _P, _I, _I, _I, _P, _I, _F, _P],
+                             _I, _I, _I, _I, _I, _P, _I, _I, _I, _P, _I, _F, _P, _P],
     "fms_sigmoid_gate": [_P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _I, _P],
     "fms_normed_add_norm": [_P, _P, _F, _P, _F, _P, _F, _P, _F, _I, _P, _F, _I, _P, _P, _F, _P, _I, _P, _I, _I, _I, _P],
     "fms_stream_mix_norm": [_P, _I, _P, _P, _P, _P, _P, _F, _P, _I, _P, _I, _I, _I, _I, _P],
     "fms_activation": [_P, _I, _I, _L, _P],
     "fms_scale_cap": [_P, _F, _F, _L, _P],
     "fms_gla_prepare": [_P, _I, _I, _I, _I, _P, _I, _P, _F, _P, _I, _P, _I, _I, _I, _F, _P],
+    "fms_gla_chunked": [_P, _I, _I, _I, _I, _P, _I, _P, _F, _F, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "fms_linear_prepare": [_P, _I, _I, _P, _I, _I, _I, _F, _I, _P],
     "fms_decay_scan": [_P, _P, _I, _I, _P, _F, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "fms_attention_prefill_sink": [_P, _P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P,
@@ -727,6 +728,9 @@ def attention_constants(head_dim: int, dtype: torch.dtype, nheads: int, kvheads:
     return _attn_constants[key]
 
 
+ROTARY_TABLE_ROWS = 256  # rows of a step from which ``qk_prepare_store`` reads the step's table of sines and cosines
+
+
 def qk_prepare_store(proj: torch.Tensor, inv_freq: Optional[torch.Tensor], rot: int, qk_norm: bool, eps: float, batch,
                      view, nheads: int, kvheads: int, dim: int, vdim: int, pad: int,
                      writes_cache: bool = True, norm_first: bool = False, q_gain: Optional[torch.Tensor] = None,
@@ -758,6 +762,8 @@ def qk_prepare_store(proj: torch.Tensor, inv_freq: Optional[torch.Tensor], rot: 
         raise KernelError(f"cache is {view.keys.dtype} with heads of {view.keys.shape[-1]}, activations are {proj.dtype}, "
                           f"heads of {pad}")
     q = None if q_in_place else torch.empty((n, nheads * pad), dtype=proj.dtype, device=proj.device)
+    # many tokens: the angles' sines and cosines come from a table that all layers with the same frequencies share
+    table = rotary_table(inv_freq, batch) if rot and n >= ROTARY_TABLE_ROWS and getattr(batch, "scratch", None) is not None else None
     _call("elementwise", "fms_qk_prepare_store", _ptr(proj), _code(proj.dtype), proj.shape[1], _ptr(q), _ptr(inv_freq),
           int(rot), float(rot_mult), 1 if qk_norm else 0, float(eps), _ptr(q_gain), _ptr(k_gain), 1 if norm_first else 0,
           1 if halves else 0,
@@ -765,7 +771,7 @@ def qk_prepare_store(proj: torch.Tensor, inv_freq: Optional[torch.Tensor], rot: 
           _ptr(batch.token_seq), _ptr(batch.slots), _ptr(view.keys), _ptr(view.values), _ptr(view.table),
           view.table.shape[1], view.block_tokens, n, nheads, kvheads, dim, vdim, pad, 1 if writes_cache else 0,
           _ptr(error_flag(proj.device)), batch.slots.shape[0], view.table.shape[0], view.keys.shape[0], first_ptr,
-          first_stride or 0, float(v_mix), _stream())
+          first_stride or 0, float(v_mix), _ptr(table), _stream())
     return q
 
 
@@ -955,6 +961,10 @@ def delta_rule_scan(qkv: torch.Tensor, proj: torch.Tensor, beta_offset: int, a_r
     return o
 
 
+GLA_CHUNKS_FROM = 32  # tokens of a sequence in one step from which its scan runs chunk by chunk
+_gla_chunk = None
+
+
 def gla_scan(proj: torch.Tensor, state: torch.Tensor, batch, heads: int, dim: int, vdim: int, rank_offset: int,
              decay_weight: torch.Tensor, decay_bias: torch.Tensor, tau: float, q_scale: float,
              writes_state: bool = True) -> torch.Tensor:
@@ -962,7 +972,9 @@ def gla_scan(proj: torch.Tensor, state: torch.Tensor, batch, heads: int, dim: in
     o = S^T (q_scale q), a = sigmoid(decay_weight u + decay_bias)^(1 / tau).  The columns of ``proj`` are [q: heads x dim |
     k: heads x dim | v: heads x vdim | ...], u its columns ``rank_offset .. rank_offset + rank``; ``decay_weight``
     [heads * dim, rank], ``decay_bias`` float32 [heads * dim]; ``state`` float32 [slots, heads, vdim, dim].  Returns o float32
-    [tokens, heads * vdim]."""
+    [tokens, heads * vdim].  Steps that bring ``GLA_CHUNKS_FROM`` tokens or more of a sequence run in chunks of tokens, others
+    token by token."""
+    global _gla_chunk, launches
     n = proj.shape[0]
     cols, channels = heads * (2 * dim + vdim), heads * dim
     rank = decay_weight.shape[1]
@@ -970,12 +982,26 @@ def gla_scan(proj: torch.Tensor, state: torch.Tensor, batch, heads: int, dim: in
         raise KernelError("gla_scan: proj [tokens, q | k | v | ... | u ...], state float32 [slots, heads, vdim, dim]")
     if decay_weight.shape[0] != channels or decay_bias.dtype != torch.float32 or decay_bias.shape[0] != channels:
         raise KernelError("gla_scan: a row of the decays' matrix and a float32 bias for every head and key channel")
+    o = torch.empty((n, heads * vdim), dtype=torch.float32, device=proj.device)
+    if batch.max_new >= GLA_CHUNKS_FROM:
+        lib = load_library("gla_chunked")
+        if _gla_chunk is None:
+            lib.fms_gla_record_floats.restype = _L
+            _gla_chunk = int(lib.fms_gla_chunk_tokens())
+        chunk_rows, first_chunk = batch.row_chunks(_gla_chunk)
+        n_chunks = chunk_rows.shape[0]
+        records = torch.empty((n_chunks * heads * int(lib.fms_gla_record_floats(dim, vdim)),), dtype=torch.float32, device=proj.device)
+        _call("gla_chunked", "fms_gla_chunked", _ptr(proj), _code(proj.dtype), proj.shape[1], int(rank_offset), rank, _ptr(decay_weight),
+              _code(decay_weight.dtype), _ptr(decay_bias), float(tau), float(q_scale), _ptr(chunk_rows), _ptr(first_chunk), n_chunks,
+              _ptr(records), _ptr(state), _ptr(o), _ptr(batch.slots), n, batch.n_seqs, heads, dim, vdim, 1 if writes_state else 0,
+              state.shape[0], _ptr(error_flag(proj.device)), _stream())
+        launches += 1
+        return o
     qkv = torch.empty((n, cols), dtype=torch.float32, device=proj.device)
     decay = torch.empty((n, channels), dtype=torch.float32, device=proj.device)
     _call("state_scan", "fms_gla_prepare", _ptr(proj), _code(proj.dtype), proj.shape[1], int(rank_offset), rank, _ptr(decay_weight),
           _code(decay_weight.dtype), _ptr(decay_bias), float(tau), _ptr(decay), channels, _ptr(qkv), n, cols, channels,
           float(q_scale), _stream())
-    o = torch.empty((n, heads * vdim), dtype=torch.float32, device=proj.device)
     _call("state_scan", "fms_decay_scan", _ptr(qkv), None, _code(proj.dtype), 0, None, 0.0, _ptr(decay), None, None, _ptr(state),
           None, _ptr(o), _ptr(batch.first_row), _ptr(batch.slots), n, batch.n_seqs, heads, dim, vdim,
           1 if writes_state else 0, state.shape[0], _stream())
@@ -1092,7 +1118,7 @@ ROUTE_SIGMOID, ROUTE_SOFTMAX, ROUTE_SIGMOID_GROUPS, ROUTE_SOFTMAX_CHOSEN = 0, 1,
 
 def route(x: torch.Tensor, router: torch.Tensor, top: int, mode: int = ROUTE_SIGMOID,
           correction: Optional[torch.Tensor] = None, route_scale: float = 1.0, groups: int = 1, keep: int = 1,
-          bias: Optional[torch.Tensor] = None, side: bool = False) -> Routing:
+          bias: Optional[torch.Tensor] = None, side: bool = False, experts: Optional[int] = None) -> Routing:
     """``ROUTE_SIGMOID``: scores sigmoid(x router^T) in float32; every token's ``top`` best experts; rows
     weight * x[token] sorted by expert.  ``ROUTE_SOFTMAX``: scores softmax(x router^T) over all experts; the ``top``
     experts with the largest score + ``correction`` [experts] (float32, or None) are the token's; its weights are their
@@ -1103,14 +1129,16 @@ def route(x: torch.Tensor, router: torch.Tensor, top: int, mode: int = ROUTE_SIG
     the correction) times ``route_scale``, and multiply the results as with ``ROUTE_SOFTMAX``.  ``ROUTE_SOFTMAX_CHOSEN``: the
     ``top`` largest logits are chosen, the weights are the softmax over those alone times ``route_scale``, and multiply the
     results.  ``bias`` [experts] float32 is added to the logits first.  ``side``: the router's matrix has a row behind the
-    experts' and ``Routing.side`` [tokens] float32 = sigmoid(x . that row), which ``route_gather`` takes for a unit that
+    experts' (``experts`` says how many those are where further rows follow) and ``Routing.side`` [tokens] float32 = sigmoid(x . that row), which ``route_gather`` takes for a unit that
     every token uses."""
-    if bias is not None and (bias.dtype != torch.float32 or bias.shape[0] != router.shape[0] - (1 if side else 0)):
+    experts = int(experts) if experts is not None else router.shape[0] - (1 if side else 0)
+    if experts + (1 if side else 0) > router.shape[0]:
+        raise KernelError(f"route: {experts} experts and {router.shape[0]} rows of the router")
+    if bias is not None and (bias.dtype != torch.float32 or bias.shape[0] != experts):
         raise KernelError("route: the bias is float32, one number an expert")
-    if correction is not None and (correction.dtype != torch.float32 or correction.shape[0] != router.shape[0] - (1 if side else 0)):
+    if correction is not None and (correction.dtype != torch.float32 or correction.shape[0] != experts):
         raise KernelError("route: the correction is float32, one number an expert")
     n, dim = x.shape
-    experts = router.shape[0] - (1 if side else 0)
     dev = x.device
     r = Routing()
     r.top, r.experts = top, experts
@@ -1134,7 +1162,7 @@ def route(x: torch.Tensor, router: torch.Tensor, top: int, mode: int = ROUTE_SIG
     _call("grouped", "fms_route", _ptr(x), _code(x.dtype), _ptr(router), _code(router.dtype), _ptr(r.expert),
           _ptr(r.weight), _ptr(counts), _ptr(r.offsets), _ptr(r.tile_first), _ptr(r.row_of_pair), _ptr(r.group_of_row),
           _ptr(r.rows), n, dim, experts, top, int(mode), _ptr(correction), float(route_scale), int(groups), int(keep),
-          _ptr(logits), _ptr(bias), _ptr(r.side), _stream())
+          _ptr(logits), router.shape[0], _ptr(bias), _ptr(r.side), _stream())
     global launches
     launches += 2
     return r

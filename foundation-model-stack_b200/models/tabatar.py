@@ -34,6 +34,7 @@ import torch
 
 from ..config.model_config import ModelConfig
 from ..config.specs import BlockSpec, DecoderSpec, FeedForwardSpec, LayerCall, MixerSpec, NormSpec, PositionSpec
+from ..parts.experts import RoutedExperts
 from ..parts.linear_attention import GatedLinearAttention
 from ..weights.adapters import register_adapter, register_adapter_step
 from ..weights.sources import TensorLayout
@@ -331,7 +332,9 @@ def _native_to_engine(tensors: Dict[str, torch.Tensor], config: TabatarConfig = 
         else:
             _fuse(held, joint, out, p + "mix.in_proj.weight")
         if mlp.get("kind") == "moe":
-            _fuse(held, ["mlp.router"] + (["mlp.shared.sg"] if _shared_ff(mlp) else []), out, p + "mlp.router.weight")
+            n, gate = int(mlp["router"].get("experts") or 0), bool(_shared_ff(mlp))
+            _fuse(held, ["mlp.router"] + (["mlp.shared.sg"] if gate else []), out, p + "mlp.router.weight",
+                  RoutedExperts.router_rows(n, gate))
             _fuse(held, ["mlp.shared.gate", "mlp.shared.up"], out, p + "mlp.shared.wg1_fused.weight")
             experts: Dict[int, Dict[str, torch.Tensor]] = {}
             for k in list(held):

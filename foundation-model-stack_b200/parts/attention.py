@@ -181,12 +181,15 @@ class SinkAttention(Part):
     def finalize(self, device, dtype) -> None:
         super().finalize(device, dtype)
         if self.rot_dims:
-            from .position import rotary_inverse_frequencies, rotary_multiplier
+            from .position import _frequencies_on_device, rotary_inverse_frequencies, rotary_multiplier
 
-            # every frequency in float64, rounded to float32 once
-            f = rotary_inverse_frequencies(self.rot_dims, float(self.position_spec.theta), self.position_spec.scaling_dict(),
-                                           dtype=torch.float64)
-            self._inv_freq = f.to(torch.float32).to(device).contiguous()
+            # every frequency in float64, rounded to float32 once; one device tensor for all layers with the same ones
+            key = ("float64", self.rot_dims, self.position_spec, str(torch.device(device)))
+            if key not in _frequencies_on_device:
+                f = rotary_inverse_frequencies(self.rot_dims, float(self.position_spec.theta), self.position_spec.scaling_dict(),
+                                               dtype=torch.float64)
+                _frequencies_on_device[key] = f.to(torch.float32).to(device).contiguous()
+            self._inv_freq = _frequencies_on_device[key]
             self.rot_mult = rotary_multiplier(self.position_spec.scaling_dict())
         if self.has_sink:
             self._sink = self.tensor("sink").float().contiguous()

@@ -30,7 +30,7 @@ Further options, each of which leaves the above as it is when absent:
     ``shared`` spec           a further unit that runs for every token: a ``projected_unit``, whose products the block makes
                               with its mixer's, or a feed-forward of its own, whose output is added here
     ``shared_gate``           the latter's output is multiplied by sigmoid(w h), one number a token; w is the row of the
-                              router's matrix behind the experts' rows (the router's product makes both)
+                              router's matrix behind the experts' rows (the router's product makes both; ``router_rows``)
 """
 from __future__ import annotations
 
@@ -76,7 +76,7 @@ class RoutedExperts(Part):
         self.in_rows = shared.in_rows if shared else 0
         self.joint_hidden, self.activation = (shared.hidden, shared.activation) if shared else (0, 0)
         self.gated = shared.gated if shared else False
-        self.router = self.add("router", Linear(spec.dim, self.experts + (1 if self.shared_gate else 0), False))
+        self.router = self.add("router", Linear(spec.dim, self.router_rows(self.experts, self.shared_gate), False))
         self.has_bias = bool(o.get("router_bias", False))
         if self.has_bias:
             self.declare("router_bias", (self.experts,), role="vector")
@@ -88,6 +88,12 @@ class RoutedExperts(Part):
             self.declare("gate_up", (self.experts, 2 * self.hidden, spec.dim), role="matrix")
         self.declare("down", (self.experts, spec.dim, self.hidden), role="matrix")
         self._correction = self._bias = None
+
+    @staticmethod
+    def router_rows(experts: int, shared_gate: bool) -> int:
+        """Rows of the router's matrix: what a checkpoint adapter has to put together ([router; shared gate; zeros up to a
+        multiple of 8, so that the library's product finds its rows aligned])."""
+        return (experts + 1 + 7) // 8 * 8 if shared_gate else experts
 
     def finalize(self, device, dtype) -> None:
         super().finalize(device, dtype)
@@ -107,7 +113,7 @@ class RoutedExperts(Part):
 
     def _routed(self, x):
         every = self.shared.forward(x) if self.shared is not None else None
-        mode, further = self._ROUTE_MODES[self.scoring], {"bias": self._bias, "side": self.shared_gate}
+        mode, further = self._ROUTE_MODES[self.scoring], {"bias": self._bias, "side": self.shared_gate, "experts": self.experts}
         if self.scoring == "sigmoid":
             routing = ops.route(x, self.router.tensor("weight"), self.top, mode, **further)
         else:

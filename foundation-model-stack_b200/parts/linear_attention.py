@@ -173,6 +173,9 @@ class GatedLinearAttention(_DecayedStateMixer):
         y = ops.gated_group_rmsnorm(o, proj, self.gate_col, ops.GATE_SILU_AFTER, self._norm, self.eps, self.vdim, proj.dtype)
         return self.dense.forward(y)
 
+    def kernel_libraries(self, dtype):
+        return super().kernel_libraries(dtype) + ["gla_chunked"]
+
 
 register_mixer("gla", GatedLinearAttention)
 register_mixer("lightning_attention", LightningAttention)
