@@ -1204,7 +1204,7 @@ FMS_API int fms_parts_group_rmsnorm(float* residual, const void* d0, float s0, c
 //   q_out null: the queries stay where they are (heads that need nothing done are read from the projection itself)
 //   q -> q_out[t, head, 0..pad) ; k, v -> the cache row of the token's slot and place, each `pad` wide:
 //   values beyond dim (vdim) are zeros, so that kernels built for one head size `pad` serve both
-// A warp per (token, head), four a block; float32 arithmetic.
+// A warp per (token, head); float32 arithmetic.
 // ---------------------------------------------------------------------------------------------------
 constexpr int PREP_MAX_PAIRS = 256;
 
@@ -1235,7 +1235,7 @@ __global__ void qk_prepare_store_kernel(const T* proj, int stride, T* q_out, con
   }
   __syncthreads();
   const int lane = threadIdx.x & 31;
-  const int item = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5) + (q_out ? 0 : nheads);  // a warp per head
+  const int item0 = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5) + (q_out ? 0 : nheads);  // a warp per head
   const T* row = proj + (size_t)t * stride;
   T* krow = nullptr;
   T* vrow = nullptr;
@@ -1255,7 +1255,7 @@ __global__ void qk_prepare_store_kernel(const T* proj, int stride, T* q_out, con
       }
     }
   }
-  if (item < nheads + 2 * kvheads) {
+  auto prepare = [&](int item) {
     if (item >= nheads + kvheads) {  // a value head: copied and padded
       const int h = item - nheads - kvheads;
       if (vrow == nullptr) return;
@@ -1374,6 +1374,106 @@ __global__ void qk_prepare_store_kernel(const T* proj, int stride, T* q_out, con
       dst[b] = from_f32<T>((sc[i].y * x1 + sc[i].x * x0) * inv);
     }
     for (int e = rot + lane; e < pad; e += 32) dst[e] = from_f32<T>(e < dim ? to_f32(src[e]) * inv : 0.f);
+  };
+  for (int item = item0; item < nheads + 2 * kvheads; item += gridDim.y * (blockDim.x >> 5)) prepare(item);
+}
+
+// The same for many bfloat16 tokens whose heads are normed first and then turned whole, in halves, with keys, values and cache
+// of one size: half / 4 lanes a head (a power of two), four pairs a lane, two heads a lane on their way at once, a block a token.
+constexpr int PREP_HALVES_THREADS = 256;
+
+__global__ void __launch_bounds__(PREP_HALVES_THREADS) qk_prepare_halves_kernel(
+    const __nv_bfloat16* proj, int stride, __nv_bfloat16* q_out, const float2* sincos, float rot_mult, int qk_norm, float eps,
+    const float* q_gain, const float* k_gain, int v_from_k, const int* positions, const int* token_seq, const int* slots,
+    __nv_bfloat16* k_cache, __nv_bfloat16* v_cache, const int* table, int table_stride, int block_tokens, int nheads, int kvheads,
+    int dim, int write_cache, int* error_flag, int n_seqs, int table_rows, int pool_blocks) {
+  pdl_launch_dependents();
+  const int half = dim >> 1, lanes = half >> 2;  // lanes of a head
+  const int sub = threadIdx.x % lanes, i = 4 * sub;
+  const int heads_at_once = blockDim.x / lanes, first = threadIdx.x / lanes;
+  float g[2][8];  // gains of queries and of keys: weights, read ahead of the wait
+#pragma unroll
+  for (int w = 0; w < 2; ++w) {
+    const float* gain = w ? k_gain : q_gain;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      g[w][k] = gain ? gain[i + k] : 1.f;
+      g[w][4 + k] = gain ? gain[half + i + k] : 1.f;
+    }
+  }
+  pdl_wait();
+  const int t = blockIdx.x;
+  const int pos = __ldcg(positions + t);
+  const __nv_bfloat16* row = proj + (size_t)t * stride;
+  float sn[4], cs[4];
+  {
+    const float4 a = *reinterpret_cast<const float4*>(sincos + (size_t)t * half + i), b = *reinterpret_cast<const float4*>(sincos + (size_t)t * half + i + 2);
+    sn[0] = a.x * rot_mult, cs[0] = a.y * rot_mult, sn[1] = a.z * rot_mult, cs[1] = a.w * rot_mult;
+    sn[2] = b.x * rot_mult, cs[2] = b.y * rot_mult, sn[3] = b.z * rot_mult, cs[3] = b.w * rot_mult;
+  }
+  size_t at = 0;
+  bool cached = false;
+  if (write_cache) {
+    const int seq = token_seq[t];
+    if (FMS_IN(seq, n_seqs)) {
+      const int slot = __ldcg(slots + seq);
+      if (FMS_IN(slot, table_rows) && FMS_IN(pos / block_tokens, table_stride)) {
+        const int blk = table[(size_t)slot * table_stride + pos / block_tokens];
+        if (blk < 0) {
+          if (threadIdx.x == 0 && error_flag) atomicExch(error_flag, 2);
+        } else if (FMS_IN(blk, pool_blocks)) {
+          cached = true;
+          at = ((size_t)blk * kvheads * block_tokens + (pos % block_tokens)) * dim;
+        }
+      }
+    }
+  }
+  const int items = nheads + 2 * kvheads;
+  for (int base = 0; base < items; base += 2 * heads_at_once) {
+    float x[2][8];
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int item = base + u * heads_at_once + first;
+#pragma unroll
+      for (int k = 0; k < 8; ++k) x[u][k] = 0.f;
+      if (item < items) {
+        const __nv_bfloat16* src = row + (size_t)(v_from_k && item >= nheads + kvheads ? item - kvheads : item) * dim;
+        float a[4], b[4];
+        ldv4(src + i, a);
+        ldv4(src + half + i, b);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) x[u][k] = a[k], x[u][4 + k] = b[k];
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int item = base + u * heads_at_once + first;
+      const bool is_q = item < nheads, is_v = item >= nheads + kvheads;
+      float ss = 0.f;
+#pragma unroll
+      for (int k = 0; k < 8; ++k) ss = fmaf(x[u][k], x[u][k], ss);
+      for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);  // every lane of the warp
+      if (item >= items) continue;
+      float a[4], b[4];
+      if (is_v) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) a[k] = x[u][k], b[k] = x[u][4 + k];
+      } else {
+        const float inv = qk_norm ? 1.f / sqrtf(ss / (float)dim + eps) : 1.f;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const float x0 = x[u][k] * inv * (is_q ? g[0][k] : g[1][k]), x1 = x[u][4 + k] * inv * (is_q ? g[0][4 + k] : g[1][4 + k]);
+          a[k] = cs[k] * x0 - sn[k] * x1;
+          b[k] = cs[k] * x1 + sn[k] * x0;
+        }
+      }
+      __nv_bfloat16* dst;
+      if (is_q) dst = q_out + ((size_t)t * nheads + item) * dim;
+      else if (!cached) continue;
+      else dst = (is_v ? v_cache : k_cache) + at + (size_t)(item - nheads - (is_v ? kvheads : 0)) * block_tokens * dim;
+      stv4(dst + i, a);
+      stv4(dst + half + i, b);
+    }
   }
 }
 
@@ -1398,8 +1498,20 @@ FMS_API int fms_qk_prepare_store(const void* proj, int dtype, int stride, void* 
                   (uintptr_t)v_cache % (4 * item) == 0 && (uintptr_t)v_first % (4 * item) == 0 && (uintptr_t)q_gain % 16 == 0 &&
                   (uintptr_t)k_gain % 16 == 0;
   const int items = (q_out ? nheads : 0) + 2 * kvheads;
+  const int lanes = dim / 8;
+  if (dtype == FMS_BF16 && vec && sincos && (uintptr_t)sincos % 16 == 0 && norm_first && halves && q_out && !v_first && rot == dim &&
+      dim == pad && dim == vdim && dim % 8 == 0 && lanes <= 32 && (lanes & (lanes - 1)) == 0) {
+    fms_launch(qk_prepare_halves_kernel, dim3(n_tokens), dim3(PREP_HALVES_THREADS), 0, stream, (const __nv_bfloat16*)proj, stride,
+               (__nv_bfloat16*)q_out, (const float2*)sincos, rot_mult, qk_norm, eps, q_gain, k_gain, v_from_k, positions, token_seq, slots,
+               (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, table, table_stride, block_tokens, nheads, kvheads, dim, write_cache,
+               error_flag, n_seqs, table_rows, pool_blocks);
+    return fms_launch_status("qk_prepare_store");
+  }
+  // few tokens: a warp a head; many: a block takes all heads of its token, so that the token's angles and its place in the
+  // cache are looked up once
+  const dim3 grid(n_tokens, n_tokens >= 592 ? 1 : (items + 3) / 4), block(n_tokens >= 592 ? 256 : 128);
   FMS_DISPATCH_DTYPE(dtype, T,
-                     fms_launch(qk_prepare_store_kernel<T>, dim3(n_tokens, (items + 3) / 4), dim3(128), 0, stream,
+                     fms_launch(qk_prepare_store_kernel<T>, grid, block, 0, stream,
                                 (const T*)proj, stride,
                                 (T*)q_out, inv_freq, rot, rot_mult, qk_norm, eps, q_gain, k_gain, norm_first, halves, v_from_k,
                                 positions, position_ids, token_seq, slots,

@@ -14,7 +14,7 @@
 //                       (fma.rn.f32x2), the column sums over channels go through a reduce-scatter of four lanes and
 //                       shared memory; records come by bulk copies (cp.async.bulk on mbarriers), several chunks ahead
 //
-// Record (floats), DP = the key size rounded up to 32, VP = the value size rounded up to VB, rows beyond a chunk's tokens and
+// Record (floats), DP = the key size rounded up to 32, 64, 128 or 256, VP = the value size rounded up to VB, rows beyond a chunk's tokens and
 // columns beyond the sizes zero (decays one):
 //   [exp(b) q: C x DP][exp(b_C - b) k: C x DP][exp(b_C): DP][A transposed, (s, t): C x C][v: VP / VB runs of C x VB]
 #include "common.cuh"
@@ -26,50 +26,69 @@ constexpr int STAGES = 3;
 
 __device__ __forceinline__ size_t record_floats(int DP, int VP) { return (size_t)2 * C * DP + DP + C * C + (size_t)C * VP; }
 
-__device__ __forceinline__ float softplus_f(float v) { return v > 0.f ? v + log1pf(expf(-v)) : log1pf(expf(v)); }
+__device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+
+// `bytes` of a row to shared memory, 16 at a time where `vec` (rows and sizes of 16 bytes), else value by value
+__device__ __forceinline__ void copy16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+// n rows of `count` values (stride `stride`) into rows of `row` values, the rows beyond n up to C zero
+template <typename T> __device__ __forceinline__ void stage_tile(T* dst, int row, const T* src, size_t stride, int n, int count, bool vec) {
+  if (vec) {
+    constexpr int PER = 16 / (int)sizeof(T);
+    const int pieces = count / PER;
+    for (int i = threadIdx.x; i < C * pieces; i += PREP_THREADS) {
+      const int t = i / pieces, c = (i - t * pieces) * PER;
+      if (t < n) copy16(dst + t * row + c, src + t * stride + c);
+      else *reinterpret_cast<uint4*>(dst + t * row + c) = make_uint4(0, 0, 0, 0);
+    }
+  } else {
+    for (int i = threadIdx.x; i < C * count; i += PREP_THREADS) {
+      const int t = i / count, c = i - t * count;
+      dst[t * row + c] = t < n ? src[t * stride + c] : from_f32<T>(0.f);
+    }
+  }
+}
 
 // chunk_rows [chunks, 2]: first row and end of every chunk.  w [heads * dim, rank], bias float32 [heads * dim].
 template <typename T, typename TW>
 __global__ void __launch_bounds__(PREP_THREADS) gla_chunk_prepare_kernel(const T* proj, int stride, int u_col, int rank, const TW* w,
                                                                          const float* bias, float inv_tau, const int* chunk_rows,
                                                                          float* records, int heads, int dim, int vdim, int DP,
-                                                                         int VP, int VB, float q_scale, int n_tokens) {
+                                                                         int VP, int VB, float q_scale, int n_tokens, int vec_qk,
+                                                                         int vec_v) {
   extern __shared__ __align__(16) float sm[];
   const int KS = DP + 4;                // padded rows of k: threads of a warp read different ones
   float* qs = sm;                       // [C][DP]
   float* as = qs + C * DP;              // [C][DP]
   float* ks = as + C * DP;              // [C][KS]
   float* us = ks + C * KS;              // [C][rank], rank rounded up to 4
-  const int RP = (rank + 3) & ~3;
+  const int RP = (rank + 3) & ~3, VR = (vdim + 7) & ~7;
+  T* rq = reinterpret_cast<T*>(us + C * RP);  // the projection's values: [C][DP] of q, of k, [C][VR] of v
+  T* rk = rq + C * DP;
+  T* rv = rk + C * DP;
   pdl_launch_dependents();
   pdl_wait();
   const int chunk = blockIdx.x, head = blockIdx.y, tid = threadIdx.x;
   const int r0 = __ldcg(chunk_rows + 2 * chunk), n = min(__ldcg(chunk_rows + 2 * chunk + 1) - r0, C);
   if (!FMS_IN(r0, n_tokens) || !FMS_IN(r0 + n - 1, n_tokens)) return;  // the whole block alike
   float* rec = records + ((size_t)chunk * heads + head) * record_floats(DP, VP);
+  const T* qp = proj + (size_t)r0 * stride + (size_t)head * dim;
+  stage_tile(rq, DP, qp, stride, n, dim, vec_qk);
+  stage_tile(rk, DP, qp + (size_t)heads * dim, stride, n, dim, vec_qk);
+  stage_tile(rv, VR, proj + (size_t)r0 * stride + 2 * (size_t)heads * dim + (size_t)head * vdim, stride, n, vdim, vec_v);
   for (int i = tid; i < C * RP; i += PREP_THREADS) {
     const int t = i / RP, r = i - t * RP;
     us[i] = t < n && r < rank ? to_f32(proj[(size_t)(r0 + t) * stride + u_col + r]) : 0.f;
   }
-  {  // v: runs of VB columns, each C x VB
-    const T* src = proj + (size_t)r0 * stride + 2 * (size_t)heads * dim + (size_t)head * vdim;
-    float* dst = rec + 2 * C * DP + DP + C * C;
-    const int per = VP / 4, vb_log = VB == 32 ? 5 : 4;
-    for (int i = tid; i < C * per; i += PREP_THREADS) {
-      const int t = i / per, v = (i - t * per) * 4;
-      float x[4];
-#pragma unroll
-      for (int k = 0; k < 4; ++k) x[k] = t < n && v + k < vdim ? to_f32(src[(size_t)t * stride + v + k]) : 0.f;
-      *reinterpret_cast<float4*>(dst + ((size_t)(v >> vb_log) * C + t) * VB + (v & (VB - 1))) = make_float4(x[0], x[1], x[2], x[3]);
-    }
-  }
+  asm volatile("cp.async.commit_group;\ncp.async.wait_group 0;\n" ::: "memory");
   __syncthreads();
   for (int d = tid; d < DP; d += PREP_THREADS) {
-    float b[C];
+    float b[C];  // ln a_t, then its sums
+#pragma unroll
+    for (int t = 0; t < C; ++t) b[t] = 0.f;
     if (d < dim) {
       const TW* row = w + ((size_t)head * dim + d) * rank;
-#pragma unroll
-      for (int t = 0; t < C; ++t) b[t] = 0.f;
       for (int r = 0; r < RP; r += 4) {
         float wv[4];
 #pragma unroll
@@ -82,29 +101,36 @@ __global__ void __launch_bounds__(PREP_THREADS) gla_chunk_prepare_kernel(const T
       }
       const float bd = bias[(size_t)head * dim + d];
 #pragma unroll
-      for (int t = 0; t < C; ++t) b[t] = t < n ? -softplus_f(-(b[t] + bd)) * inv_tau : 0.f;  // ln a_t
-    } else {
-#pragma unroll
-      for (int t = 0; t < C; ++t) b[t] = 0.f;
+      for (int t = 0; t < C; ++t) b[t] = t < n ? -softplus_f(-(b[t] + bd)) * inv_tau : 0.f;
     }
-    const T* qp = proj + (size_t)r0 * stride + (size_t)head * dim + d;
-    const T* kp = qp + (size_t)heads * dim;
-    float kv[C], sum = 0.f;
+    float sum = 0.f;
 #pragma unroll
     for (int t = 0; t < C; ++t) {
       as[t * DP + d] = expf(b[t]);
       sum += b[t];
       b[t] = sum;
-      const bool in = t < n && d < dim;
-      const float q = in ? to_f32(qp[(size_t)t * stride]) * q_scale : 0.f;
-      kv[t] = in ? to_f32(kp[(size_t)t * stride]) : 0.f;
+      const float q = d < dim ? to_f32(rq[t * DP + d]) * q_scale : 0.f;
       qs[t * DP + d] = q;
-      ks[t * KS + d] = kv[t];
       rec[t * DP + d] = q * expf(sum);
     }
 #pragma unroll
-    for (int t = 0; t < C; ++t) rec[(C + t) * DP + d] = kv[t] * expf(sum - b[t]);
+    for (int t = 0; t < C; ++t) {
+      const float k = d < dim ? to_f32(rk[t * DP + d]) : 0.f;
+      ks[t * KS + d] = k;
+      rec[(C + t) * DP + d] = k * expf(sum - b[t]);
+    }
     rec[2 * C * DP + d] = expf(sum);
+  }
+  {  // v: runs of VB columns, each C x VB
+    float* dst = rec + 2 * C * DP + DP + C * C;
+    const int per = VP / 4, vb_log = VB == 32 ? 5 : 4;
+    for (int i = tid; i < C * per; i += PREP_THREADS) {
+      const int t = i / per, v = (i - t * per) * 4;
+      float x[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) x[k] = v + k < vdim ? to_f32(rv[t * VR + v + k]) : 0.f;
+      *reinterpret_cast<float4*>(dst + ((size_t)(v >> vb_log) * C + t) * VB + (v & (VB - 1))) = make_float4(x[0], x[1], x[2], x[3]);
+    }
   }
   __syncthreads();
   // A: thread (s, run of channels); k_s carries the product of the decays after s
@@ -164,18 +190,20 @@ __device__ __forceinline__ Eight load8(const float* x) {  // shared memory, 16-b
 
 // Block: WD = DP / 32 warps along the channels x VB / 16 along the value columns.  A lane holds channels d0 .. d0 + 8 of
 // columns v0, v0 + 1.  state [slots, heads, vdim, dim]; o [tokens, heads * vdim].
-__global__ void __launch_bounds__(512, 1) gla_chunk_scan_kernel(const float* records, const int* chunk_rows, const int* first_chunk,
+template <int DP, int VB>
+__global__ void __launch_bounds__(DP / 32 * (VB / 16) * 32) gla_chunk_scan_kernel(const float* records, const int* chunk_rows, const int* first_chunk,
                                                              float* state, float* o, const int* slots, int heads, int dim, int vdim,
-                                                             int DP, int VP, int VB, int write_state, int n_slots, int n_tokens,
+                                                             int VP, int write_state, int n_slots, int n_tokens,
                                                              int* error_flag) {
   extern __shared__ __align__(16) float sm[];
   __shared__ __align__(8) unsigned long long full[STAGES];
   pdl_launch_dependents();
   const int seq = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int WD = DP / 32, wd = warp % WD, wv = warp / WD;
+  constexpr int WD = DP / 32;
+  const int wd = warp % WD, wv = warp / WD;
   const int dgl = lane >> 3, vgl = lane & 7, dg = wd * 4 + dgl;
   const int d0 = dg * 8, vl = wv * 16 + vgl * 2, v0 = blockIdx.z * VB + vl;
-  const int head_part = 2 * C * DP + DP + C * C, stage_floats = head_part + C * VB;
+  constexpr int head_part = 2 * C * DP + DP + C * C, stage_floats = head_part + C * VB;
   float* red = sm + STAGES * stage_floats;  // [2][WD][C][VB]
   if (tid == 0) {
     for (int i = 0; i < STAGES; ++i) mbar_init(full + i, 1);
@@ -186,6 +214,8 @@ __global__ void __launch_bounds__(512, 1) gla_chunk_scan_kernel(const float* rec
   if (!FMS_IN(slot, n_slots)) return;  // the whole block alike
   const int c_lo = __ldcg(first_chunk + seq), c_hi = __ldcg(first_chunk + seq + 1);
   const size_t rec_floats = record_floats(DP, VP);
+  const int first_row = c_lo < c_hi ? __ldcg(chunk_rows + 2 * c_lo) : 0;  // a sequence's chunks follow one another
+  const int end_row = c_lo < c_hi ? __ldcg(chunk_rows + 2 * c_hi - 1) : 0;
   auto issue = [&](int c) {  // one thread
     const int st = (c - c_lo) % STAGES;
     const float* rec = records + ((size_t)c * heads + head) * rec_floats;
@@ -211,7 +241,7 @@ __global__ void __launch_bounds__(512, 1) gla_chunk_scan_kernel(const float* rec
   bool dead = false;  // a copy did not come in time: the block goes on with what lies there, and says so
   for (int c = c_lo; c < c_hi; ++c) {
     const int i = c - c_lo, st = i % STAGES;
-    const int row0 = __ldcg(chunk_rows + 2 * c), rows = min(__ldcg(chunk_rows + 2 * c + 1) - row0, C);
+    const int row0 = first_row + i * C, rows = min(end_row - row0, C);
     if (!dead && !mbar_wait(full + st, (i / STAGES) & 1)) dead = true;
     const float* Q = sm + st * stage_floats;
     const float* K = Q + C * DP;
@@ -221,10 +251,13 @@ __global__ void __launch_bounds__(512, 1) gla_chunk_scan_kernel(const float* rec
     float* mine = red + (size_t)(i & 1) * WD * C * VB;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
+      // r[t]: token half * 8 + (t ^ turn), so that what a lane keeps and what it hands on below are the same places of r
+      // in every lane
       float r[8][2];
+      const int turn = 2 * dgl;
 #pragma unroll
       for (int t = 0; t < 8; ++t) {
-        const Eight q = load8(Q + (half * 8 + t) * DP + d0);
+        const Eight q = load8(Q + (half * 8 + (t & 1)) * DP + ((t ^ turn) & 6) * DP + d0);
         f32x2 a0 = mul2(q.p[0], S[0][0]), a1 = mul2(q.p[0], S[0][1]);
 #pragma unroll
         for (int j = 1; j < 4; ++j) {
@@ -240,30 +273,24 @@ __global__ void __launch_bounds__(512, 1) gla_chunk_scan_kernel(const float* rec
       // the chunk's own tokens: every group of channels takes its share of the s
       for (int s = dg; s < C; s += 4 * WD) {
         const float2 v = *reinterpret_cast<const float2*>(V + s * VB + vl);
-        const float4 x = *reinterpret_cast<const float4*>(AT + s * C + half * 8), y = *reinterpret_cast<const float4*>(AT + s * C + half * 8 + 4);
-        const float a[8] = {x.x, x.y, x.z, x.w, y.x, y.y, y.z, y.w};
 #pragma unroll
-        for (int t = 0; t < 8; ++t) {
-          r[t][0] = fmaf(a[t], v.x, r[t][0]);
-          r[t][1] = fmaf(a[t], v.y, r[t][1]);
+        for (int t = 0; t < 8; t += 2) {
+          const float2 a = *reinterpret_cast<const float2*>(AT + s * C + half * 8 + (t ^ turn));
+          r[t][0] = fmaf(a.x, v.x, r[t][0]);
+          r[t][1] = fmaf(a.x, v.y, r[t][1]);
+          r[t + 1][0] = fmaf(a.y, v.x, r[t + 1][0]);
+          r[t + 1][1] = fmaf(a.y, v.y, r[t + 1][1]);
         }
       }
       // over the four lanes of a column pair: lane dgl ends with tokens 2 dgl and 2 dgl + 1
-      const bool hi = dgl & 2, odd = dgl & 1;
 #pragma unroll
       for (int t = 0; t < 4; ++t)
 #pragma unroll
-        for (int k = 0; k < 2; ++k) {
-          const float other = __shfl_xor_sync(0xffffffffu, hi ? r[t][k] : r[t + 4][k], 16);
-          r[t][k] = (hi ? r[t + 4][k] : r[t][k]) + other;
-        }
+        for (int k = 0; k < 2; ++k) r[t][k] += __shfl_xor_sync(0xffffffffu, r[t + 4][k], 16);
 #pragma unroll
       for (int t = 0; t < 2; ++t)
 #pragma unroll
-        for (int k = 0; k < 2; ++k) {
-          const float other = __shfl_xor_sync(0xffffffffu, odd ? r[t][k] : r[t + 2][k], 8);
-          r[t][k] = (odd ? r[t + 2][k] : r[t][k]) + other;
-        }
+        for (int k = 0; k < 2; ++k) r[t][k] += __shfl_xor_sync(0xffffffffu, r[t + 2][k], 8);
 #pragma unroll
       for (int t = 0; t < 2; ++t)
         *reinterpret_cast<float2*>(mine + ((size_t)wd * C + half * 8 + 2 * dgl + t) * VB + vl) = make_float2(r[t][0], r[t][1]);
@@ -329,18 +356,16 @@ __global__ void __launch_bounds__(512, 1) gla_chunk_scan_kernel(const float* rec
   }
 }
 
-int padded_dim(int dim) { return (dim + 31) / 32 * 32; }
-int value_run(int dim, int vdim) {  // value columns of a block: at most 512 threads
-  return vdim > 16 && padded_dim(dim) / 32 * 2 * 32 <= 512 ? 32 : 16;
-}
-int padded_vdim(int dim, int vdim) { return (vdim + value_run(dim, vdim) - 1) / value_run(dim, vdim) * value_run(dim, vdim); }
+int padded_dim(int dim) { return dim <= 32 ? 32 : (dim <= 64 ? 64 : (dim <= 128 ? 128 : 256)); }
+int value_run(int vdim) { return vdim > 16 ? 32 : 16; }  // value columns of a block
+int padded_vdim(int vdim) { return (vdim + value_run(vdim) - 1) / value_run(vdim) * value_run(vdim); }
 }  // namespace
 
 FMS_API int fms_gla_chunk_tokens() { return C; }
 // floats of one (chunk, head)'s record
 FMS_API long fms_gla_record_floats(int dim, int vdim) {
   const long DP = padded_dim(dim);
-  return 2L * C * DP + DP + C * C + (long)C * padded_vdim(dim, vdim);
+  return 2L * C * DP + DP + C * C + (long)C * padded_vdim(vdim);
 }
 
 // proj: rows of `stride` values, [q: heads x dim | k: heads x dim | v: heads x vdim | ...], u at columns u_col .. u_col + rank;
@@ -355,22 +380,39 @@ FMS_API int fms_gla_chunked(const void* proj, int dtype, int stride, int u_col, 
   if (heads <= 0 || heads > 65535 || dim <= 0 || dim > 256 || vdim <= 0 || rank <= 0 || rank > 1024 || !(tau > 0.f))
     return fms_fail("gla_chunked: %d heads, dim %d (up to 256), vdim %d, rank %d (up to 1024), tau %f", heads, dim, vdim, rank, tau);
   if ((uintptr_t)records % 16 || (uintptr_t)o % 8) return fms_fail("gla_chunked: scratch and results must be aligned");
-  const int DP = padded_dim(dim), VB = value_run(dim, vdim), VP = padded_vdim(dim, vdim);
-  const size_t prep = ((size_t)3 * C * DP + C * 4 + (size_t)C * ((rank + 3) & ~3)) * sizeof(float);
+  const int DP = padded_dim(dim), VB = value_run(vdim), VP = padded_vdim(vdim);
+  const size_t item = dtype == FMS_BF16 ? 2 : 4;
+  const size_t prep = ((size_t)3 * C * DP + C * 4 + (size_t)C * ((rank + 3) & ~3)) * sizeof(float) +
+                      (size_t)C * (2 * DP + ((vdim + 7) & ~7)) * item;
+  // 16-byte copies: every row of a head's values starts on 16 bytes and its size is a multiple of them
+  const bool rows16 = (uintptr_t)proj % 16 == 0 && (size_t)stride * item % 16 == 0;
+  const int vec_qk = rows16 && (size_t)dim * item % 16 == 0;
+  const int vec_v = rows16 && (size_t)vdim * item % 16 == 0 && (size_t)2 * heads * dim * item % 16 == 0;
   const size_t prep_smem = prep > 4 * C * C * sizeof(float) ? prep : 4 * C * C * sizeof(float);
   FMS_DISPATCH_DTYPE(dtype, T, FMS_DISPATCH_DTYPE(w_dtype, TW, {
     if (prep_smem > 48 * 1024)
       cudaFuncSetAttribute(gla_chunk_prepare_kernel<T, TW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prep_smem);
     fms_launch(gla_chunk_prepare_kernel<T, TW>, dim3(n_chunks, heads), dim3(PREP_THREADS), prep_smem, stream, (const T*)proj, stride,
                u_col, rank, (const TW*)w, bias, (float)(1.0 / (double)tau), chunk_rows, records, heads, dim, vdim, DP, VP, VB, q_scale,
-               n_tokens);
+               n_tokens, vec_qk, vec_v);
   }));
   if (fms_launch_status("gla_chunk_prepare")) return 1;
-  const int WD = DP / 32, WV = VB / 16;
-  const size_t smem = ((size_t)STAGES * (2 * C * DP + DP + C * C + C * VB) + (size_t)2 * WD * C * VB) * sizeof(float);
-  if (smem > 220 * 1024) return fms_fail("gla_chunked: %zu bytes of shared memory", smem);
-  cudaFuncSetAttribute(gla_chunk_scan_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  fms_launch(gla_chunk_scan_kernel, dim3(n_seqs, heads, VP / VB), dim3(32 * WD * WV), smem, stream, (const float*)records, chunk_rows,
-             first_chunk, state, o, slots, heads, dim, vdim, DP, VP, VB, write_state, n_slots, n_tokens, error_flag);
+#define FMS_GLA_SCAN(DP_, VB_)                                                                                              \
+  do {                                                                                                                      \
+    constexpr size_t smem = ((size_t)STAGES * (2 * C * DP_ + DP_ + C * C + C * VB_) + (size_t)2 * (DP_ / 32) * C * VB_) * sizeof(float); \
+    static_assert(smem <= 220 * 1024, "stages and sums fit shared memory");                                                 \
+    cudaFuncSetAttribute(gla_chunk_scan_kernel<DP_, VB_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
+    fms_launch(gla_chunk_scan_kernel<DP_, VB_>, dim3(n_seqs, heads, VP / VB), dim3(DP_ / 32 * (VB_ / 16) * 32), smem, stream, \
+               (const float*)records, chunk_rows, first_chunk, state, o, slots, heads, dim, vdim, VP, write_state, n_slots,  \
+               n_tokens, error_flag);                                                                                        \
+  } while (0)
+  if (VB == 32) {
+    if (DP == 32) FMS_GLA_SCAN(32, 32); else if (DP == 64) FMS_GLA_SCAN(64, 32);
+    else if (DP == 128) FMS_GLA_SCAN(128, 32); else FMS_GLA_SCAN(256, 32);
+  } else {
+    if (DP == 32) FMS_GLA_SCAN(32, 16); else if (DP == 64) FMS_GLA_SCAN(64, 16);
+    else if (DP == 128) FMS_GLA_SCAN(128, 16); else FMS_GLA_SCAN(256, 16);
+  }
+#undef FMS_GLA_SCAN
   return fms_launch_status("gla_chunk_scan");
 }
