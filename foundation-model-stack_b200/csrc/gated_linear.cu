@@ -1,6 +1,13 @@
-// Gated linear attention over many tokens of a sequence, chunk by chunk.  Per head, with one decay a token and key channel:
+// Gated linear attention.  Per head, with one decay a token and key channel:
 //   S_t = diag(a_t) S_(t-1) + k_t v_t^T;   o_t = S_t^T q_t;   a = sigmoid(W u + bias)^(1 / tau)
-// (state_scan.cu walks the same recurrence token by token: decode steps and short portions.)  A chunk is C tokens of one
+// Here are the kernels for many tokens of a sequence, chunk by chunk, and for a decode step, which has one token of every
+// sequence (state_scan.cu walks the same recurrence token by token: short portions, and sizes that these do not take).
+//
+//   gla_decode          a block per (sequence, head): the state's rows are asked for first, all of a warp's at once; then the
+//                       decays, the update, the read-out, the head's root mean square, its weight and the silu gate, in one
+//                       kernel between the two projections
+//
+// Many tokens.  A chunk is C tokens of one
 // sequence's rows of the step, from the step's first row on.  With b_t = ln a_1 + .. + ln a_t inside a chunk that starts at S:
 //   o_t = S^T (exp(b_t) q_t) + sum_(s <= t) A[t, s] v_s         A[t, s] = sum_d q_t[d] k_s[d] a_(s+1)[d] .. a_t[d]
 //   S'  = diag(exp(b_C)) S + sum_s (exp(b_C - b_s) k_s) v_s^T
@@ -356,6 +363,129 @@ __global__ void __launch_bounds__(DP / 32 * (VB / 16) * 32) gla_chunk_scan_kerne
   }
 }
 
+// ---- a decode step ---------------------------------------------------------------------------------------
+// L lanes hold a row of the state (a value column's dim key channels, 4 * N a lane); a warp takes 32 / L rows at once and
+// ROWS such groups a tile.
+constexpr int DECODE_WARPS = 8;
+
+// sums r[0 .. COUNT) over the L lanes of a row by halves: a lane ends with the row whose number is returned, in r[0]
+template <int COUNT, int L> __device__ __forceinline__ int rows_sum(float (&r)[COUNT], int lane) {
+  int row = 0, half = COUNT;
+#pragma unroll
+  for (int o = L / 2; o > 0; o >>= 1) {
+    if (half > 1) {
+      half >>= 1;
+      const bool hi = lane & o;
+#pragma unroll
+      for (int j = 0; j < COUNT / 2; ++j) {
+        if (j < half) {
+          const float other = __shfl_xor_sync(0xffffffffu, hi ? r[j] : r[j + half], o);
+          r[j] = (hi ? r[j + half] : r[j]) + other;
+        }
+      }
+      if (hi) row += half;
+    } else {
+      r[0] += __shfl_xor_sync(0xffffffffu, r[0], o);
+    }
+  }
+  return row;
+}
+
+// proj: a row a sequence, [q: heads x dim | k | v: heads x vdim | ...], u at u_col, the gates' logits at gate_col;
+// out [rows, heads * vdim] = o / sqrt(mean over the head(o^2) + eps) * norm[vdim] * silu(gate)
+template <typename T, typename TW, int L, int N>
+__global__ void __launch_bounds__(32 * DECODE_WARPS, 2) gla_decode_kernel(const T* proj, int stride, int u_col, int rank, const TW* w,
+                                                                       const float* bias, double inv_tau, float q_scale, float* state,
+                                                                       const int* slots, int gate_col, const float* norm, float eps, T* out,
+                                                                       int heads, int dim, int vdim, int write_state, int n_slots) {
+  constexpr int ROWS = N == 1 ? L / 2 : 8, PER = 32 / L;  // 16 rows a warp and tile (N == 2: 8)
+  extern __shared__ __align__(16) float sm[];  // [rank]
+  __shared__ __align__(16) float qs[256], ks[256], as[256];
+  __shared__ float scratch[33];
+  float* os = sm + ((rank + 3) & ~3);  // [vdim]
+  float* vs = os + vdim;               // [vdim]
+  pdl_launch_dependents();
+  pdl_wait();
+  const int seq = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int slot = __ldcg(slots + seq);
+  if (!FMS_IN(slot, n_slots)) return;  // the whole block alike
+  const T* row = proj + (size_t)seq * stride;
+  float* st = state + ((size_t)slot * heads + head) * vdim * dim;
+  const int sub = lane / L, at = (lane % L) * 4;  // the lane's row within a group and its first channel
+  float4 S[ROWS][N];
+  auto load = [&](int base) {
+#pragma unroll
+    for (int j = 0; j < ROWS; ++j) {
+      const int v = base + j * PER + sub;
+#pragma unroll
+      for (int e = 0; e < N; ++e)
+        S[j][e] = v < vdim && at + e * 4 * L < dim ? __ldcg(reinterpret_cast<const float4*>(st + (size_t)v * dim + at + e * 4 * L)) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  };
+  load(warp * ROWS * PER);
+  for (int r = tid; r < rank; r += blockDim.x) sm[r] = to_f32(row[u_col + r]);
+  for (int d = tid; d < 256; d += blockDim.x) {
+    qs[d] = d < dim ? to_f32(row[(size_t)head * dim + d]) * q_scale : 0.f;
+    ks[d] = d < dim ? to_f32(row[(size_t)(heads + head) * dim + d]) : 0.f;
+  }
+  for (int v = tid; v < vdim; v += blockDim.x) vs[v] = to_f32(row[2 * (size_t)heads * dim + (size_t)head * vdim + v]);
+  __syncthreads();
+  for (int d = tid; d < 256; d += blockDim.x) {
+    float a = 0.f;
+    if (d < dim) {
+      const TW* wr = w + ((size_t)head * dim + d) * rank;
+      float z = bias[(size_t)head * dim + d], z2 = 0.f;
+      int r = 0;
+#pragma unroll 4
+      for (; r + 1 < rank; r += 2) {
+        z = fmaf(to_f32(wr[r]), sm[r], z);
+        z2 = fmaf(to_f32(wr[r + 1]), sm[r + 1], z2);
+      }
+      if (r < rank) z = fmaf(to_f32(wr[r]), sm[r], z);
+      // taken in double and rounded once: a decay's error compounds over a sequence
+      const double m = -(double)(z + z2);
+      a = (float)exp(-(m > 40.0 ? m : log1p(exp(m))) * inv_tau);
+    }
+    as[d] = a;
+  }
+  __syncthreads();
+  float4 q[N], k[N], a[N];
+#pragma unroll
+  for (int e = 0; e < N; ++e) {
+    q[e] = *reinterpret_cast<const float4*>(qs + at + e * 4 * L);
+    k[e] = *reinterpret_cast<const float4*>(ks + at + e * 4 * L);
+    a[e] = *reinterpret_cast<const float4*>(as + at + e * 4 * L);
+  }
+  for (int base = warp * ROWS * PER; base < vdim; base += DECODE_WARPS * ROWS * PER) {  // the whole warp alike
+    if (base != warp * ROWS * PER) load(base);
+    float r[ROWS];
+#pragma unroll
+    for (int j = 0; j < ROWS; ++j) {
+      const int v = base + j * PER + sub;
+      const float x = v < vdim ? vs[v] : 0.f;
+      r[j] = 0.f;
+#pragma unroll
+      for (int e = 0; e < N; ++e) {
+        float4 s = S[j][e];
+        s.x = fmaf(a[e].x, s.x, k[e].x * x), s.y = fmaf(a[e].y, s.y, k[e].y * x);
+        s.z = fmaf(a[e].z, s.z, k[e].z * x), s.w = fmaf(a[e].w, s.w, k[e].w * x);
+        r[j] += fmaf(s.x, q[e].x, s.y * q[e].y) + fmaf(s.z, q[e].z, s.w * q[e].w);
+        if (write_state && v < vdim && at + e * 4 * L < dim) *reinterpret_cast<float4*>(st + (size_t)v * dim + at + e * 4 * L) = s;
+      }
+    }
+    const int mine = base + rows_sum<ROWS, L>(r, lane) * PER + sub;
+    if (mine < vdim) os[mine] = r[0];  // lanes that end with the same row write the same sum
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int v = tid; v < vdim; v += blockDim.x) ss = fmaf(os[v], os[v], ss);
+  const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)vdim + eps);
+  for (int v = tid; v < vdim; v += blockDim.x) {
+    const float g = to_f32(row[gate_col + (size_t)head * vdim + v]);
+    out[((size_t)seq * heads + head) * vdim + v] = from_f32<T>(os[v] * inv * norm[v] * (g / (1.f + expf(-g))));
+  }
+}
+
 int padded_dim(int dim) { return dim <= 32 ? 32 : (dim <= 64 ? 64 : (dim <= 128 ? 128 : 256)); }
 int value_run(int vdim) { return vdim > 16 ? 32 : 16; }  // value columns of a block
 int padded_vdim(int vdim) { return (vdim + value_run(vdim) - 1) / value_run(vdim) * value_run(vdim); }
@@ -415,4 +545,27 @@ FMS_API int fms_gla_chunked(const void* proj, int dtype, int stride, int u_col, 
   }
 #undef FMS_GLA_SCAN
   return fms_launch_status("gla_chunk_scan");
+}
+
+// One token of every sequence: row i of proj belongs to the sequence in slots[i].  norm [vdim] float32; out [n_seqs, heads * vdim]
+// in proj's dtype.  dim a multiple of 4, state 16-byte aligned.
+FMS_API int fms_gla_decode(const void* proj, int dtype, int stride, int u_col, int rank, const void* w, int w_dtype, const float* bias,
+                           float tau, float q_scale, float* state, const int* slots, int gate_col, const float* norm, float eps, void* out,
+                           int n_seqs, int heads, int dim, int vdim, int write_state, int n_slots, cudaStream_t stream) {
+  if (n_seqs <= 0) return 0;
+  if (heads <= 0 || heads > 65535 || dim <= 0 || dim > 256 || dim % 4 || vdim <= 0 || vdim > 4096 || rank <= 0 || rank > 1024 || !(tau > 0.f) ||
+      (uintptr_t)state % 16)
+    return fms_fail("gla_decode: %d heads, dim %d (a multiple of 4 up to 256), vdim %d, rank %d (up to 1024), tau %f", heads, dim, vdim, rank, tau);
+  const size_t smem = (size_t)(((rank + 3) & ~3) + 2 * vdim) * sizeof(float);
+#define FMS_GLA_DECODE(L, N)                                                                                                \
+  FMS_DISPATCH_DTYPE(dtype, T, FMS_DISPATCH_DTYPE(w_dtype, TW,                                                              \
+                     fms_launch(gla_decode_kernel<T, TW, L, N>, dim3(n_seqs, heads), dim3(32 * DECODE_WARPS), smem, stream,  \
+                                (const T*)proj, stride, u_col, rank, (const TW*)w, bias, 1.0 / (double)tau, q_scale, state,  \
+                                slots, gate_col, norm, eps, (T*)out, heads, dim, vdim, write_state, n_slots)))
+  if (dim <= 32) FMS_GLA_DECODE(8, 1);
+  else if (dim <= 64) FMS_GLA_DECODE(16, 1);
+  else if (dim <= 128) FMS_GLA_DECODE(32, 1);
+  else FMS_GLA_DECODE(32, 2);
+#undef FMS_GLA_DECODE
+  return fms_launch_status("gla_decode");
 }

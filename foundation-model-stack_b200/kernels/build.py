@@ -41,7 +41,7 @@ PLAIN_LIBRARIES = {
     "sampling": ("sampling.cu", []),
     "recurrent": ("recurrent.cu", []),
     "state_scan": ("state_scan.cu", []),
-    "gla_chunked": ("gla_chunked.cu", []),
+    "gated_linear": ("gated_linear.cu", []),
     "grouped": ("grouped.cu", []),
     "latent_attention": ("latent_attention.cu", []),
 }

@@ -87,6 +87,7 @@ _SIGNATURES = {
     "fms_scale_cap": [_P, _F, _F, _L, _P],
     "fms_gla_prepare": [_P, _I, _I, _I, _I, _P, _I, _P, _F, _P, _I, _P, _I, _I, _I, _F, _P],
     "fms_gla_chunked": [_P, _I, _I, _I, _I, _P, _I, _P, _F, _F, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
+    "fms_gla_decode": [_P, _I, _I, _I, _I, _P, _I, _P, _F, _F, _P, _P, _I, _P, _F, _P, _I, _I, _I, _I, _I, _I, _P],
     "fms_linear_prepare": [_P, _I, _I, _P, _I, _I, _I, _F, _I, _P],
     "fms_decay_scan": [_P, _P, _I, _I, _P, _F, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "fms_attention_prefill_sink": [_P, _P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P,
@@ -984,14 +985,14 @@ def gla_scan(proj: torch.Tensor, state: torch.Tensor, batch, heads: int, dim: in
         raise KernelError("gla_scan: a row of the decays' matrix and a float32 bias for every head and key channel")
     o = torch.empty((n, heads * vdim), dtype=torch.float32, device=proj.device)
     if batch.max_new >= GLA_CHUNKS_FROM:
-        lib = load_library("gla_chunked")
+        lib = load_library("gated_linear")
         if _gla_chunk is None:
             lib.fms_gla_record_floats.restype = _L
             _gla_chunk = int(lib.fms_gla_chunk_tokens())
         chunk_rows, first_chunk = batch.row_chunks(_gla_chunk)
         n_chunks = chunk_rows.shape[0]
         records = torch.empty((n_chunks * heads * int(lib.fms_gla_record_floats(dim, vdim)),), dtype=torch.float32, device=proj.device)
-        _call("gla_chunked", "fms_gla_chunked", _ptr(proj), _code(proj.dtype), proj.shape[1], int(rank_offset), rank, _ptr(decay_weight),
+        _call("gated_linear", "fms_gla_chunked", _ptr(proj), _code(proj.dtype), proj.shape[1], int(rank_offset), rank, _ptr(decay_weight),
               _code(decay_weight.dtype), _ptr(decay_bias), float(tau), float(q_scale), _ptr(chunk_rows), _ptr(first_chunk), n_chunks,
               _ptr(records), _ptr(state), _ptr(o), _ptr(batch.slots), n, batch.n_seqs, heads, dim, vdim, 1 if writes_state else 0,
               state.shape[0], _ptr(error_flag(proj.device)), _stream())
@@ -1006,6 +1007,28 @@ def gla_scan(proj: torch.Tensor, state: torch.Tensor, batch, heads: int, dim: in
           None, _ptr(o), _ptr(batch.first_row), _ptr(batch.slots), n, batch.n_seqs, heads, dim, vdim,
           1 if writes_state else 0, state.shape[0], _stream())
     return o
+
+
+def gla_read_out(proj: torch.Tensor, state: torch.Tensor, batch, heads: int, dim: int, vdim: int, rank_offset: int,
+                 decay_weight: torch.Tensor, decay_bias: torch.Tensor, tau: float, q_scale: float, gate_offset: int, norm: torch.Tensor,
+                 eps: float, writes_state: bool = True) -> torch.Tensor:
+    """``gla_scan`` and what follows it: every head divided by its root mean square, times ``norm`` (float32 [vdim]), times
+    silu of ``proj``'s columns from ``gate_offset`` on; [tokens, heads * vdim] in proj's dtype.  A decode step (one token of
+    every sequence) is one kernel, else the scan and ``gated_group_rmsnorm``."""
+    n = proj.shape[0]
+    if batch.decode and dim % 4 == 0 and vdim <= 4096 and n == batch.n_seqs:
+        rank = decay_weight.shape[1]
+        if state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, vdim, dim) or norm.dtype != torch.float32 or norm.shape[0] != vdim \
+                or proj.shape[1] < max(heads * (2 * dim + vdim), rank_offset + rank, gate_offset + heads * vdim) \
+                or decay_weight.shape[0] != heads * dim or decay_bias.dtype != torch.float32 or decay_bias.shape[0] != heads * dim:
+            raise KernelError("gla_read_out: proj [tokens, q | k | v | ...], state float32 [slots, heads, vdim, dim], norm float32 [vdim]")
+        out = torch.empty((n, heads * vdim), dtype=proj.dtype, device=proj.device)
+        _call("gated_linear", "fms_gla_decode", _ptr(proj), _code(proj.dtype), proj.shape[1], int(rank_offset), rank, _ptr(decay_weight),
+              _code(decay_weight.dtype), _ptr(decay_bias), float(tau), float(q_scale), _ptr(state), _ptr(batch.slots), int(gate_offset),
+              _ptr(norm), float(eps), _ptr(out), n, heads, dim, vdim, 1 if writes_state else 0, state.shape[0], _stream())
+        return out
+    o = gla_scan(proj, state, batch, heads, dim, vdim, rank_offset, decay_weight, decay_bias, tau, q_scale, writes_state)
+    return gated_group_rmsnorm(o, proj, gate_offset, GATE_SILU_AFTER, norm, eps, vdim, proj.dtype)
 
 
 ACT_NONE, ACT_SILU = 0, 1

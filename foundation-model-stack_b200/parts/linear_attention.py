@@ -168,13 +168,13 @@ class GatedLinearAttention(_DecayedStateMixer):
 
     def forward(self, x, batch, cache_view, writes_cache: bool = True):
         proj = self.in_proj.forward(x)
-        o = ops.gla_scan(proj, cache_view.state, batch, self.heads, self.head_dim, self.vdim, self.rank_col,
-                         self.decay_out.tensor("weight"), self._decay_bias, self.tau, self.head_dim ** -0.5, writes_cache)
-        y = ops.gated_group_rmsnorm(o, proj, self.gate_col, ops.GATE_SILU_AFTER, self._norm, self.eps, self.vdim, proj.dtype)
+        y = ops.gla_read_out(proj, cache_view.state, batch, self.heads, self.head_dim, self.vdim, self.rank_col,
+                             self.decay_out.tensor("weight"), self._decay_bias, self.tau, self.head_dim ** -0.5, self.gate_col, self._norm,
+                             self.eps, writes_cache)
         return self.dense.forward(y)
 
     def kernel_libraries(self, dtype):
-        return super().kernel_libraries(dtype) + ["gla_chunked"]
+        return super().kernel_libraries(dtype) + ["gated_linear"]
 
 
 register_mixer("gla", GatedLinearAttention)
