@@ -71,10 +71,11 @@ __global__ void __launch_bounds__(PREP_THREADS) gla_chunk_prepare_kernel(const T
   float* ks = as + C * DP;              // [C][KS]
   float* us = ks + C * KS;              // [C][rank], rank rounded up to 4
   const int RP = (rank + 3) & ~3, VR = (vdim + 7) & ~7;
+  // no early launch of the kernel that follows: the scan has about a block a multiprocessor, and started while these blocks
+  // still fill most of them, its blocks would crowd on the few that are free
   T* rq = reinterpret_cast<T*>(us + C * RP);  // the projection's values: [C][DP] of q, of k, [C][VR] of v
   T* rk = rq + C * DP;
   T* rv = rk + C * DP;
-  pdl_launch_dependents();
   pdl_wait();
   const int chunk = blockIdx.x, head = blockIdx.y, tid = threadIdx.x;
   const int r0 = __ldcg(chunk_rows + 2 * chunk), n = min(__ldcg(chunk_rows + 2 * chunk + 1) - r0, C);
@@ -531,8 +532,10 @@ FMS_API int fms_gla_chunked(const void* proj, int dtype, int stride, int u_col, 
   do {                                                                                                                      \
     constexpr size_t smem = ((size_t)STAGES * (2 * C * DP_ + DP_ + C * C + C * VB_) + (size_t)2 * (DP_ / 32) * C * VB_) * sizeof(float); \
     static_assert(smem <= 220 * 1024, "stages and sums fit shared memory");                                                 \
-    cudaFuncSetAttribute(gla_chunk_scan_kernel<DP_, VB_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
-    fms_launch(gla_chunk_scan_kernel<DP_, VB_>, dim3(n_seqs, heads, VP / VB), dim3(DP_ / 32 * (VB_ / 16) * 32), smem, stream, \
+    cudaFuncSetAttribute(gla_chunk_scan_kernel<DP_, VB_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(smem < 116 * 1024 ? 116 * 1024 : smem)); \
+    /* up to a block a multiprocessor: as much shared memory as keeps a second one away */                                  \
+    const size_t want = (long)n_seqs * heads * (VP / VB) <= 148 && smem < 116 * 1024 ? 116 * 1024 : smem;                    \
+    fms_launch(gla_chunk_scan_kernel<DP_, VB_>, dim3(n_seqs, heads, VP / VB), dim3(DP_ / 32 * (VB_ / 16) * 32), want, stream, \
                (const float*)records, chunk_rows, first_chunk, state, o, slots, heads, dim, vdim, VP, write_state, n_slots,  \
                n_tokens, error_flag);                                                                                        \
   } while (0)
