@@ -212,6 +212,10 @@ class Cache:
             self.groups.append(group)
             for layer in layers:
                 self._group_of_layer[layer] = group
+        self._windows = sorted({g.request.window for g in self.groups if isinstance(g, KVGroup) and g.request.window})
+        # slots whose last step brought one token: all that has left a window by then has been given back, so that the next
+        # such step has something to do only where a block begins or the first key a window keeps moves into another block
+        self._settled: set = set()
 
     # ---- slots -------------------------------------------------------------------------------
     def begin(self, n: int, first_positions: Optional[Sequence[int]] = None) -> List[int]:
@@ -241,6 +245,7 @@ class Cache:
                     g.release(s)
             self.length[s] = 0
             self.position[s] = 0
+            self._settled.discard(s)
             self.slots.free(s)
 
     # ---- one step ----------------------------------------------------------------------------
@@ -251,6 +256,7 @@ class Cache:
         if len(set(slots)) != len(slots):
             raise ValueError("a slot appears twice in one step")
         before = []
+        self._settled.difference_update(slots)
         for s, n in zip(slots, num_new):
             if not self.slots.is_held(s):
                 raise ValueError(f"slot {s} is not held")
@@ -281,17 +287,21 @@ class Cache:
 
     def prepare_decode(self, slots: Sequence[int]) -> None:
         """``prepare`` for a step of one token per sequence, without looking at whole table rows: a block
-        is needed only when a sequence's length is a multiple of 64, and a window only moves then."""
+        is needed only when a sequence's length is a multiple of 64, and given back only when the first key that a window
+        keeps is the first of a block (or after a step of several tokens)."""
         work = []
         for s in slots:
             n = self.length[s]
             if max(n, self.position[s]) + 1 > self.max_positions:
                 raise CacheFull(f"slot {s}: {max(n, self.position[s])} + 1 tokens exceed the model's "
                                 f"{self.max_positions} positions")
-            if n % BLOCK_TOKENS == 0 or any(isinstance(g, KVGroup) and g.request.window for g in self.groups):
+            if n % BLOCK_TOKENS == 0 or (self._windows and s not in self._settled) \
+                    or any(n >= w and (n - w + 1) % BLOCK_TOKENS == 0 for w in self._windows):
                 work.append(s)
         if work:
             self.prepare(work, [1] * len(work))
+        if self._windows:
+            self._settled.update(slots)
 
     def commit(self, slots: Sequence[int], num_new: Sequence[int]) -> None:
         for s, n in zip(slots, num_new):

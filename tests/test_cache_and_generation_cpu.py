@@ -473,3 +473,33 @@ def test_sentencepiece_model_file(tmp_path):
         pieces = tok.tokenize("the lazy fox")
         assert tok.convert_tokens_to_ids(pieces) == ids[1:] and tok.convert_tokens_to_string(pieces) == "the lazy fox"
         assert tok.convert_ids_to_tokens(ids[1:]) == pieces
+
+
+def test_decode_steps_give_back_what_has_left_a_window_as_soon_as_any_step_would():
+    """Steps of one token look at a windowed group's table only where something can have changed; after every step the
+    blocks held are those that looking every time would hold."""
+    from fms_b200.cache import Cache, KVRequest
+
+    requests = [KVRequest(1, 16, w) for w in (0, 1, 5, 64, 65, 130)]
+    quick, thorough = (Cache(requests, 64 * 40, 2048, torch.float32, "cpu", max_slots=4) for _ in range(2))
+    held = lambda c: [[(row >= 0).tolist() for row in g.table_host] for g in c.groups]
+    for prompts in ((1, 64, 200, 333), (63, 129, 300, 5)):
+        slots = quick.begin(4)
+        assert slots == thorough.begin(4)
+        for c in (quick, thorough):
+            c.prepare(slots, prompts)
+            c.commit(slots, prompts)
+        for step in range(150):
+            live = slots if step < 70 else slots[1:3]
+            if step in (40, 100):  # a portion of several tokens in between
+                for c in (quick, thorough):
+                    c.prepare(live, [70] * len(live))
+                    c.commit(live, [70] * len(live))
+            quick.prepare_decode(live)
+            thorough.prepare(live, [1] * len(live))
+            assert held(quick) == held(thorough)
+            for c in (quick, thorough):
+                c.commit(live, [1] * len(live))
+        for c in (quick, thorough):
+            c.release(slots)
+            assert all(g.pool.n_held == 0 for g in c.groups)
