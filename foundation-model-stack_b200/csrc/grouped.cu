@@ -553,7 +553,8 @@ __global__ void __launch_bounds__(128) route_scatter_kernel(const T* __restrict_
     for (int d = threadIdx.x; d < dim; d += blockDim.x) dst[d] = src[d];
 }
 
-template <typename T>
+// A block per token and run of 256 x (8 or 1) columns.  EVERY: what every token adds beside its pairs' rows.
+template <typename T, bool EVERY>
 __global__ void __launch_bounds__(256) route_gather_kernel(const T* __restrict__ ys, const int* __restrict__ row_of_pair,
                                                            T* __restrict__ out, int dim, int top, int n_pairs,
                                                            const float* weight, const T* shared, const float* side,
@@ -567,38 +568,40 @@ __global__ void __launch_bounds__(256) route_gather_kernel(const T* __restrict__
     rows_of_token[k] = ld_fresh(row_of_pair + (size_t)t * top + k);
     weight_of_token[k] = weight ? ld_fresh(weight + (size_t)t * top + k) : 1.f;
   }
-  __syncthreads();
-  const T* every = shared ? shared + (size_t)t * dim : nullptr;
-  const float gate = every && side ? ld_fresh(side + t) : 1.f;
-  if (vec) {
-    for (int d = 8 * threadIdx.x; d < dim; d += 8 * blockDim.x) {
-      float a[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-      if (every) {
-        rows_load8(every + d, a);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) a[e] *= gate;
-      }
-#pragma unroll 4
-      for (int k = 0; k < top; ++k) {
-        const int row = rows_of_token[k];
-        if (!FMS_IN(row, n_pairs)) continue;
-        float v[8];
-        rows_load8(ys + (size_t)row * dim + d, v);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) a[e] = fmaf(weight_of_token[k], v[e], a[e]);
-      }
-      rows_store8(out + (size_t)t * dim + d, a);
-    }
-    return;
+  const float gate = EVERY && side ? ld_fresh(side + t) : 1.f;
+  const int d = (vec ? 8 : 1) * (blockIdx.y * blockDim.x + threadIdx.x);
+  float s[8];
+  if (EVERY && d < dim) {  // asked for ahead of the pairs' rows, added behind them
+    if (vec) rows_load8(shared + (size_t)t * dim + d, s);
+    else s[0] = to_f32(shared[(size_t)t * dim + d]);
   }
-  for (int d = threadIdx.x; d < dim; d += blockDim.x) {
-    float a = every ? gate * to_f32(every[d]) : 0.f;
+  __syncthreads();
+  if (d >= dim) return;
+  if (vec) {
+    float a[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
     for (int k = 0; k < top; ++k) {
       const int row = rows_of_token[k];
-      if (FMS_IN(row, n_pairs)) a = fmaf(weight_of_token[k], to_f32(ys[(size_t)row * dim + d]), a);
+      if (!FMS_IN(row, n_pairs)) continue;
+      float v[8];
+      rows_load8(ys + (size_t)row * dim + d, v);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) a[e] = fmaf(weight_of_token[k], v[e], a[e]);
     }
-    out[(size_t)t * dim + d] = from_f32<T>(a);
+    if (EVERY) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) a[e] = fmaf(gate, s[e], a[e]);
+    }
+    rows_store8(out + (size_t)t * dim + d, a);
+    return;
   }
+  float a = 0.f;
+  for (int k = 0; k < top; ++k) {
+    const int row = rows_of_token[k];
+    if (FMS_IN(row, n_pairs)) a = fmaf(weight_of_token[k], to_f32(ys[(size_t)row * dim + d]), a);
+  }
+  if (EVERY) a = fmaf(gate, s[0], a);
+  out[(size_t)t * dim + d] = from_f32<T>(a);
 }
 }  // namespace
 
@@ -761,9 +764,15 @@ FMS_API int fms_gated_clamped(const void* gu, void* out, int dtype, int n_rows, 
 FMS_API int fms_route_gather(const void* ys, int dtype, const int* row_of_pair, void* out, int n_tokens, int dim, int top,
                              const float* weight, const void* shared, const float* side, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
-  FMS_DISPATCH_DTYPE(dtype, T,
-                     fms_launch(route_gather_kernel<T>, dim3(n_tokens), dim3(256), 2 * sizeof(int) * top, stream, (const T*)ys, row_of_pair,
-                                (T*)out, dim, top, n_tokens * top, weight, (const T*)shared, side,
-                                dim % 8 == 0 && (((uintptr_t)ys | (uintptr_t)out | (uintptr_t)shared) & 15) == 0 ? 1 : 0));
+  const int vec = dim % 8 == 0 && (((uintptr_t)ys | (uintptr_t)out | (uintptr_t)shared) & 15) == 0 ? 1 : 0;
+  const dim3 grid(n_tokens, (dim + (vec ? 8 : 1) * 256 - 1) / ((vec ? 8 : 1) * 256));
+  FMS_DISPATCH_DTYPE(dtype, T, {
+    if (shared)
+      fms_launch(route_gather_kernel<T, true>, grid, dim3(256), 2 * sizeof(int) * top, stream, (const T*)ys, row_of_pair, (T*)out, dim,
+                 top, n_tokens * top, weight, (const T*)shared, side, vec);
+    else
+      fms_launch(route_gather_kernel<T, false>, grid, dim3(256), 2 * sizeof(int) * top, stream, (const T*)ys, row_of_pair, (T*)out, dim,
+                 top, n_tokens * top, weight, (const T*)nullptr, side, vec);
+  });
   return fms_launch_status("route_gather");
 }
